@@ -17,6 +17,7 @@ from .metanex import MetanexConfig
 from .rofulorn import RofulornConfig
 from .fuzelorn import FuzelornConfig
 from .dodilix import DodilixConfig
+from .matepel import MatepelConfig
 
 _ARCHITECTURES: Dict[str, Any] = {}
 _MODEL_TYPES: Dict[str, str] = {}
@@ -66,3 +67,4 @@ register_architecture("Metanex", MetanexConfig)
 register_architecture("Rofulorn", RofulornConfig)
 register_architecture("Fuzelorn", FuzelornConfig)
 register_architecture("Dodilix", DodilixConfig)
+register_architecture("Matepel", MatepelConfig)

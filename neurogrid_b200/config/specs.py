@@ -52,6 +52,10 @@ class RopeSpec:
     ``freq_scaling`` = (factor, low, high, original) rescales the frequencies by their wavelength l = 2 pi / f:
     f stays where l < original / high, becomes f / factor where l > original / low, and in between
     (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+    ``yarn`` = (factor, original, fast, slow) rescales them by their index instead: with
+    at(t) = dims ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(at(fast)), 0), hi = min(ceil(at(slow)), dims - 1)
+    and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), f_i becomes r_i f_i / factor + (1 - r_i) f_i; cosines and
+    sines are multiplied by 0.1 ln(factor) + 1.
     """
     head_dim: int
     theta: float
@@ -59,6 +63,7 @@ class RopeSpec:
     scale: float = 1.0
     rotary_dims: Optional[int] = None
     freq_scaling: Optional[Tuple[float, float, float, float]] = None
+    yarn: Optional[Tuple[float, float, float, float]] = None
     kind: str = "rope"
 
     def __post_init__(self):
@@ -68,6 +73,8 @@ class RopeSpec:
             raise ValueError("rope needs an even head_dim")
         if self.rotary_dims is not None and (self.rotary_dims % 2 or not 0 <= self.rotary_dims <= self.head_dim):
             raise ValueError(f"rotary_dims must be even and at most head_dim, got {self.rotary_dims}")
+        if self.yarn is not None and (self.freq_scaling is not None or min(self.yarn) <= 0 or self.theta == 1.0):
+            raise ValueError("yarn scaling: four positive numbers, a base other than 1, and no other scaling of the frequencies")
 
 
 @dataclass(frozen=True)
@@ -139,7 +146,9 @@ class MappedAttentionSpec:
     sequence's position 0 (``cache_window`` is then c: no later query reads further back).  ``norm_weight`` False: the
     RMS norm of q and k has no weights, and since a rotation keeps a head's sum of squares it may be taken on either
     side of ``position``.  ``out_gate``: the concatenated heads are multiplied element by element by the sigmoid of
-    one more projection of the mixer's input (rows ``g``) before the output projection.
+    one more projection of the mixer's input (rows ``g``) before the output projection.  ``unit_sink``: the softmax's
+    denominator holds one more 1, a sink whose score is 0 for every head (nothing is learned).  ``shared_kv``: there is
+    no v projection, the values are the keys as projected (with their bias, before norm and ``position``).
     """
     hidden: int
     n_heads: int
@@ -165,6 +174,8 @@ class MappedAttentionSpec:
     chunk: Optional[int] = None
     norm_weight: bool = True
     out_gate: bool = False
+    unit_sink: bool = False
+    shared_kv: bool = False
     names: Mapping[str, str] = field(default_factory=lambda: _names(
         q="q", k="k", v="v", o="o", q_bias="q.b", k_bias="k.b", v_bias="v.b", o_bias="o.b", q_norm="q.norm",
         k_norm="k.norm", lq1="lq1", lk1="lk1", lq2="lq2", lk2="lk2", sink="sink", out_gate="g"))
@@ -187,6 +198,12 @@ class MappedAttentionSpec:
             raise ValueError("a chunked mask has a positive size and goes without a window or kept first tokens")
         if not self.norm_weight and self.norm_scope != "head":
             raise ValueError("a norm without weights is a norm per head")
+        if self.sink and self.unit_sink:
+            raise ValueError("a softmax has one sink")
+        if self.shared_kv and (self.n_maps != 1 or self.value_dim != self.key_dim):
+            raise ValueError("values that are the keys have the keys' size and one map")
+        if self.qk_norm and not self.norm_weight and getattr(self.position, "yarn", None) is not None:
+            raise ValueError("a norm without weights goes with a rotation that keeps lengths")
 
 
 @dataclass(frozen=True)
@@ -206,7 +223,8 @@ class ShortConvSpec:
 
 @dataclass(frozen=True)
 class SwiGLUSpec:
-    """down( act(gate(x)) * up(x) ), no biases; ``activation`` "silu" or "gelu_tanh" (the tanh form of gelu).
+    """down( act(gate(x)) * up(x) ), no biases; ``activation`` "silu" or "gelu_tanh" (the tanh form of gelu), or
+    "clamped_glu": g sigmoid(``glu_alpha`` g) (u + 1) with g = min(gate(x), limit), u = clamp(up(x), -limit, limit).
     A tensor's name is its role's name plus ``weight_suffix``."""
     hidden: int
     intermediate: int
@@ -214,11 +232,15 @@ class SwiGLUSpec:
         gate="gate_proj", up="up_proj", down="down_proj"))
     activation: str = "silu"
     weight_suffix: str = ".weight"
+    limit: float = 0.0
+    glu_alpha: float = 1.702
     kind: str = "swiglu"
 
     def __post_init__(self):
-        if self.activation not in ("silu", "gelu_tanh"):
-            raise ValueError(f"gated feed-forward: activation must be silu or gelu_tanh, got {self.activation!r}")
+        if self.activation not in ("silu", "gelu_tanh", "clamped_glu"):
+            raise ValueError(f"gated feed-forward: activation must be silu, gelu_tanh or clamped_glu, got {self.activation!r}")
+        if self.activation == "clamped_glu" and not self.limit > 0:
+            raise ValueError("gated feed-forward: the clamped activation needs a positive limit")
 
 
 @dataclass(frozen=True)
@@ -409,7 +431,8 @@ class GatedDeltaSpec:
 class SideBySideSpec:
     """Two mixers that read the same input; the result is half the sum of their outputs, each first divided by its
     root mean square over the model width (``eps``) and multiplied by a plain weight of its own.
-    ``combine`` "weighted": the result is left_scale * left + right_scale * right instead (no norms, no weights)."""
+    ``combine`` "weighted": the result is left_scale * left + right_scale * right instead (no norms, no weights; a bias
+    of a side's output projection is scaled with it)."""
     hidden: int
     left: object
     right: object
@@ -450,6 +473,57 @@ class GatedLinearAttentionSpec:
     def __post_init__(self):
         if min(self.n_heads, self.key_dim, self.value_dim, self.decay_rank) < 1 or not self.tau > 0:
             raise ValueError("gated linear attention: heads, sizes and tau must be positive")
+
+
+@dataclass(frozen=True)
+class LightningSpec:
+    """Linear attention with a fixed decay per head on activated projections:
+
+        S <- decay_h S + k_t v_t^T;   o_t = S^T q_t      (S [key_dim, value_dim] per head, float32, zero at the start)
+
+    q = silu(W_q x), k = silu(W_k x) (``n_heads`` heads of ``key_dim``), v = silu(W_v x) (heads of ``value_dim``); no
+    other scale.  All heads' o together are RMS-normed (one mean over n_heads * value_dim, a plain weight of that
+    length, ``eps``), multiplied by sigmoid(W_g x) and projected back."""
+    hidden: int
+    n_heads: int
+    key_dim: int
+    value_dim: int
+    decay: Tuple[float, ...]
+    eps: float
+    names: Mapping[str, str] = field(default_factory=lambda: _names(q="q", k="k", v="v", gate="g", o="o", norm="norm"))
+    kind: str = "lightning_attention"
+
+    def __post_init__(self):
+        if min(self.n_heads, self.key_dim, self.value_dim) < 1 or self.key_dim > 512:
+            raise ValueError("lightning attention: heads and sizes must be positive, key_dim at most 512")
+        if len(self.decay) != self.n_heads or not all(0.0 <= d <= 1.0 for d in self.decay):
+            raise ValueError(f"lightning attention: {self.n_heads} decays between 0 and 1, got {self.decay}")
+
+
+@dataclass(frozen=True)
+class MLSTMSpec:
+    """The matrix memory of xLSTM: exponential gates per head and token with a running maximum m (0 at the start),
+
+        i = c tanh((W_i x + b_i) / c),  f = log sigmoid(c tanh((W_f x + b_f) / c))       (c = ``gate_cap``)
+        m' = max(f + m, i);  S <- exp(f + m - m') S + exp(i - m') k v^T;  n likewise with k alone
+        o = S^T q / (max(|n . q|, exp(-m')) + 1e-6)
+
+    q = W_q x * key_dim^(-1/2), k = W_k x (``n_heads`` heads of ``key_dim``), v = W_v x (heads of ``value_dim``).  Each
+    head's o is divided by its root mean square (``eps``), the heads are multiplied by a plain weight as long as all of
+    them and by sigmoid(W_g x), then projected back.  State per request: S, n and m, float32, zero at the start."""
+    hidden: int
+    n_heads: int
+    key_dim: int
+    value_dim: int
+    gate_cap: float
+    eps: float
+    names: Mapping[str, str] = field(default_factory=lambda: _names(
+        q="q", k="k", v="v", gate="g", o="o", norm="norm", input_gate="i", input_bias="i.b", forget_gate="f", forget_bias="f.b"))
+    kind: str = "mlstm"
+
+    def __post_init__(self):
+        if min(self.n_heads, self.key_dim, self.value_dim) < 1 or self.key_dim > 512 or not self.gate_cap > 0:
+            raise ValueError("mlstm: heads, sizes and the gates' cap must be positive, key_dim at most 512")
 
 
 @dataclass(frozen=True)
@@ -548,9 +622,13 @@ class ModelSpec:
     logit_scale: float = 1.0                     # logits <- logits * scale
     streams: int = 0                             # > 0: the residual stream is that many copies (hyper-connections); every
                                                  # layer's block arrangement then keeps them ("hyper")
+    embed_norm: Optional[object] = None          # a norm of the (scaled) embedding, float32: what the first layer reads
+    embed_norm_name: str = "embed.norm"
 
     def __post_init__(self):
         n = len(self.layers)
+        if self.embed_norm is not None and (self.position_table_name or self.token_pair is not None):
+            raise ValueError("a normed embedding goes without a position table and token pairs")
         if self.position_table_name and self.max_positions <= 0:
             raise ValueError("a table of learned positions needs max_positions")
         if self.streams < 0 or (self.streams > 0) != any(l.block == "hyper" for l in self.layers) \

@@ -47,6 +47,46 @@ NG_EXPORT int ng_embed(const void* table, int table_bf16, const int* tokens, flo
     return ng_launch_status();
 }
 
+// out[row] = e / sqrt(mean(e^2) + eps) * w with e = table[token] * scale: the embedding and the norm behind it in one
+// kernel, float32 (a block per row; the second pass reads the row from the cache again).
+template <typename T>
+__global__ void embed_norm_kernel(const T* __restrict__ table, const int* __restrict__ tokens, const float* __restrict__ w,
+                                  float* __restrict__ out, int H, int V, int* __restrict__ status, float scale, float eps) {
+    __shared__ float red[32];
+    ng_pdl_trigger();
+    ng_pdl_wait();
+    const int row = blockIdx.x;
+    const int tok = tokens[row];
+    float* dst = out + (size_t)row * H;
+    if (tok < 0 || tok >= V) {
+        if (threadIdx.x == 0) atomicOr(status, NG_STATUS_BAD_TOKEN);
+        for (int j = threadIdx.x; j < H; j += blockDim.x) dst[j] = 0.f;
+        return;
+    }
+    const T* src = table + (size_t)tok * H;
+    float ss = 0.f;
+    for (int j = threadIdx.x; j < H; j += blockDim.x) {
+        const float v = ng_ld(src + j) * scale;
+        ss = fmaf(v, v, ss);
+    }
+    const float r = rsqrtf(ng_block_sum(ss, red) / (float)H + eps);
+    for (int j = threadIdx.x; j < H; j += blockDim.x) dst[j] = ng_ld(src + j) * scale * r * w[j];
+}
+
+NG_EXPORT int ng_embed_norm(const void* table, int table_bf16, const int* tokens, const float* w, float* out, int n_rows,
+                            int H, int V, int* status, float scale, float eps, cudaStream_t stream) {
+    if (n_rows <= 0) return NG_OK;
+    if (H <= 0 || V <= 0) return NG_BAD_SIZE;
+    const int threads = H >= 1024 ? 256 : 128;
+    if (table_bf16)
+        NG_LAUNCH((embed_norm_kernel<__nv_bfloat16>), n_rows, threads, 0, stream, (const __nv_bfloat16*)table, tokens, w, out, H,
+                  V, status, scale, eps);
+    else
+        NG_LAUNCH((embed_norm_kernel<float>), n_rows, threads, 0, stream, (const float*)table, tokens, w, out, H, V, status,
+                  scale, eps);
+    return ng_launch_status();
+}
+
 // dst[i] = src[idx[i]] where idx[i] >= 0 (else dst[i] stays): tokens sampled on the device feed the
 // next step without passing through the host
 __global__ void gather_i32_kernel(int* __restrict__ dst, const int* __restrict__ src, const int* __restrict__ idx, int n) {
@@ -293,15 +333,23 @@ NG_EXPORT int ng_residual_add(float* h, const void* delta, long long n, int delt
 }
 
 // ---------------------------------------------------------------------------------- swiglu
-// gu is [n_rows, 2*I]: gate = gu[:, :I], up = gu[:, I:];  out = act(gate) * up, float32 math;
-// act: silu, or (`gelu`) the tanh form of gelu, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))).  `out` rows lie
-// `ldo` elements apart (a column block of a wider buffer).
-__device__ __forceinline__ float ng_gate_act(float g, int gelu) {
-    if (gelu) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-    return g / (1.f + expf(-g));
+// gu is [n_rows, 2*I]: gate g = gu[:, :I], up u = gu[:, I:];  out = act(g) * u, float32 math;  act 0: silu, 1: the tanh
+// form of gelu, 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))), 2: both clamped, g' sigmoid(alpha g') (u' + 1) with
+// g' = min(g, limit), u' = clamp(u, -limit, limit).  `out` rows lie `ldo` elements apart (a column block of a wider buffer).
+struct GateAct {
+    int kind;
+    float limit, alpha;
+};
+__device__ __forceinline__ float ng_gated(float g, float u, const GateAct& a) {
+    if (a.kind == 2) {
+        g = fminf(g, a.limit);
+        return g / (1.f + expf(-a.alpha * g)) * (fminf(fmaxf(u, -a.limit), a.limit) + 1.f);
+    }
+    if (a.kind == 1) return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
+    return g / (1.f + expf(-g)) * u;
 }
 template <typename T>
-__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, int ldo, int gelu) {
+__global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int I, int ldo, GateAct act) {
     ng_pdl_trigger();
     ng_pdl_wait();
     const size_t row = blockIdx.x;
@@ -309,12 +357,12 @@ __global__ void swiglu_kernel(const T* __restrict__ gu, T* __restrict__ out, int
     if (j >= I) return;
     const float g = ng_ld(gu + row * 2 * (size_t)I + j);
     const float u = ng_ld(gu + row * 2 * (size_t)I + I + j);
-    ng_st(out + row * (size_t)ldo + j, ng_gate_act(g, gelu) * u);
+    ng_st(out + row * (size_t)ldo + j, ng_gated(g, u, act));
 }
 
 // bfloat16, I % 8 == 0: eight elements (16 bytes of gate, 16 of up) per thread
 __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_bfloat16* __restrict__ out, int I, int ldo,
-                                     int gelu) {
+                                     GateAct act) {
     ng_pdl_trigger();
     ng_pdl_wait();
     const size_t row = blockIdx.x;
@@ -330,22 +378,25 @@ __global__ void swiglu_bf16x8_kernel(const __nv_bfloat16* __restrict__ gu, __nv_
     for (int k = 0; k < 4; ++k) {
         const float ga = __low2float(g2[k]), gb = __high2float(g2[k]);
         const float ua = __low2float(u2[k]), ub = __high2float(u2[k]);
-        o2[k] = __floats2bfloat162_rn(ng_gate_act(ga, gelu) * ua, ng_gate_act(gb, gelu) * ub);
+        o2[k] = __floats2bfloat162_rn(ng_gated(ga, ua, act), ng_gated(gb, ub, act));
     }
     *reinterpret_cast<uint4*>(out + row * (size_t)ldo + j) = o4;
 }
 
-NG_EXPORT int ng_swiglu(const void* gu, void* out, int n_rows, int I, int ldo, int gelu, int act_bf16, cudaStream_t stream) {
+NG_EXPORT int ng_swiglu(const void* gu, void* out, int n_rows, int I, int ldo, int kind, float limit, float alpha, int act_bf16,
+                        cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
+    const GateAct act{kind, limit, alpha};
+    if (kind < 0 || kind > 2 || (kind == 2 && !(limit > 0.f))) return NG_BAD_SIZE;
     if (I <= 0 || (I + 255) / 256 > 65535 || ldo < I) return NG_BAD_SIZE;
     if (act_bf16 && I % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)gu & 15) == 0 && ((uintptr_t)out & 15) == 0) {
         dim3 grid8(n_rows, (I / 8 + 127) / 128);
-        NG_LAUNCH((swiglu_bf16x8_kernel), grid8, 128, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, I, ldo, gelu);
+        NG_LAUNCH((swiglu_bf16x8_kernel), grid8, 128, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, I, ldo, act);
         return ng_launch_status();
     }
     dim3 grid(n_rows, (I + 255) / 256);
-    if (act_bf16) NG_LAUNCH((swiglu_kernel<__nv_bfloat16>), grid, 256, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, I, ldo, gelu);
-    else NG_LAUNCH((swiglu_kernel<float>), grid, 256, 0, stream, (const float*)gu, (float*)out, I, ldo, gelu);
+    if (act_bf16) NG_LAUNCH((swiglu_kernel<__nv_bfloat16>), grid, 256, 0, stream, (const __nv_bfloat16*)gu, (__nv_bfloat16*)out, I, ldo, act);
+    else NG_LAUNCH((swiglu_kernel<float>), grid, 256, 0, stream, (const float*)gu, (float*)out, I, ldo, act);
     return ng_launch_status();
 }
 

@@ -41,7 +41,8 @@ struct GemmParams {
                                // blocks fill the SMs evenly
     int w_bytes;               // bytes of W a stage receives (rows, or 2 * rows for SwiGLU, times 128)
     int red_v4;                // EPI_RED: four columns per atomic (N, ldc multiples of 4, out 16-byte aligned)
-    int gate_gelu;             // EPI_SWIGLU: the gate's activation is the tanh form of gelu instead of silu
+    int gate_kind;             // EPI_SWIGLU: the gate's activation, 0 silu, 1 the tanh form of gelu, 2 both halves clamped
+    float gate_limit, gate_alpha;    // ... 2: g' sigmoid(alpha g') (u' + 1), g' = min(g, limit), u' = clamp(u, -limit, limit)
     int relu2;                 // EPI_BF16: out = relu(y)^2 of the rounded y = x w^T + bias (what a separate pass over y gives)
 };
 
@@ -214,7 +215,14 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
                         // the unfused path rounds both products to bf16 before the gate: keep that rounding
                         const float g = __bfloat162float(__float2bfloat16_rn(up_half ? theirs : mine));
                         const float u = __bfloat162float(__float2bfloat16_rn(up_half ? mine : theirs));
-                        reinterpret_cast<bf16*>(p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn((p.gate_gelu ? gelu_tanh(g) : silu_fast(g)) * u);
+                        float y;
+                        if (p.gate_kind == 2) {
+                            const float gc = fminf(g, p.gate_limit);
+                            y = gc / (1.f + expf(-p.gate_alpha * gc)) * (fminf(fmaxf(u, -p.gate_limit), p.gate_limit) + 1.f);
+                        } else {
+                            y = (p.gate_kind == 1 ? gelu_tanh(g) : silu_fast(g)) * u;
+                        }
+                        reinterpret_cast<bf16*>(p.out)[(size_t)m * p.ldc + n] = __float2bfloat16_rn(y);
                     }
                 }
             }
@@ -308,15 +316,18 @@ static int dispatch_tn(int tn, const CUtensorMap& mw, const CUtensorMap& mx, con
 //   epi 3: out float [M, ldc] += x w^T (atomic adds; any splits)
 //   epi 4: as epi 2 with gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) for silu
 //   epi 5: as epi 0, then relu(.)^2 of the rounded result
+//   epi 6: as epi 2 with both halves clamped: g' sigmoid(gate_alpha g') (u' + 1), g' = min(g, gate_limit),
+//          u' = clamp(u, -gate_limit, gate_limit)
 // tn: token tile (16, 32, 64, 128, 256; 0 = chosen from M).
 NG_EXPORT int ng_gemm_sm100(const void* x, const void* w, const void* bias, void* out, int M, int N, int K,
-                            int n_w_rows, int ldc, int epi, int splits, int up_row_offset, int tn, int* status,
-                            cudaStream_t stream) {
+                            int n_w_rows, int ldc, int epi, int splits, int up_row_offset, int tn, float gate_limit,
+                            float gate_alpha, int* status, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return NG_OK;
     if (K <= 0 || K % 8 || ((uintptr_t)x & 15) || ((uintptr_t)w & 15) || ldc < N || splits < 1 || !status)
         return NG_BAD_SIZE;
-    const int gate_gelu = epi == 4, relu2 = epi == 5;
-    if (gate_gelu) epi = EPI_SWIGLU;
+    const int gate_kind = epi == 4 ? 1 : epi == 6 ? 2 : 0, relu2 = epi == 5;
+    if (gate_kind == 2 && !(gate_limit > 0.f)) return NG_BAD_SIZE;
+    if (gate_kind) epi = EPI_SWIGLU;
     if (relu2) epi = EPI_BF16;
     if (epi < 0 || epi > 3 || ((epi == EPI_BF16 || epi == EPI_SWIGLU) && splits != 1) ||
         (epi == EPI_SWIGLU && up_row_offset + N > n_w_rows))
@@ -332,7 +343,7 @@ NG_EXPORT int ng_gemm_sm100(const void* x, const void* w, const void* bias, void
     if (!tensor_map(w, n_w_rows, K, rows, &mw)) return NG_LAUNCH_FAILED;
     if (!tensor_map(x, M, K, tn, &mx)) return NG_LAUNCH_FAILED;
     const int red_v4 = epi == EPI_RED && N % 4 == 0 && ldc % 4 == 0 && rows % 4 == 0 && ((uintptr_t)out & 15) == 0;
-    GemmParams p{out, (const bf16*)bias, status, M, N, K, ldc, per, up_row_offset, rows, w_bytes, red_v4, gate_gelu, relu2};
+    GemmParams p{out, (const bf16*)bias, status, M, N, K, ldc, per, up_row_offset, rows, w_bytes, red_v4, gate_kind, gate_limit, gate_alpha, relu2};
     dim3 grid((N + rows - 1) / rows, (M + tn - 1) / tn, splits);
     if (grid.y > 65535 || grid.z > 65535) return NG_BAD_SIZE;
     switch (epi) {

@@ -7,6 +7,7 @@
 //   2. with `delta` (the output y of the sublayer before: [n, H] of the activation type, or float32 partial sums that
 //      are added in ascending order) all streams are replaced at once from the old ones,
 //          x_t <- sum_s mix[s, t] x_s + out_w[t] * y            (mix is indexed [from, to]);
+//      `bias` [H] (float32, optional) belongs to y: it is added to delta's value;
 //   3. with `in_w`: u = sum_t in_w[t] x_t is what the next sublayer reads, and `out` receives
 //      u / sqrt(mean(u^2) + eps) * norm_w in the activation type (one rounding);
 //   4. with `sum_out`: the sum of the streams (float32 [n, H]), which is what the model's last norm reads.
@@ -22,7 +23,7 @@ __global__ void __launch_bounds__(512)
 hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __restrict__ delta, int n_partials,
                size_t partial_stride, const float* __restrict__ mix, const float* __restrict__ out_w,
                const float* __restrict__ in_w, const float* __restrict__ norm_w, TO* __restrict__ out,
-               float* __restrict__ sum_out, int S_rt, int H, float eps) {
+               float* __restrict__ sum_out, const float* __restrict__ bias, int S_rt, int H, float eps) {
     extern __shared__ float u_s[];                     // [H]: what the next sublayer reads, before its norm
     __shared__ float red[32];
     __shared__ float mix_s[HC_MAX_STREAMS * HC_MAX_STREAMS], ow_s[HC_MAX_STREAMS], iw_s[HC_MAX_STREAMS];
@@ -72,6 +73,7 @@ hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __
             for (int v = 0; v < VEC; ++v) {
                 y[v] = 0.f;
                 for (int p = 0; p < n_partials; ++p) y[v] += ng_ld(delta + p * partial_stride + row * H + j + v);   // ascending p
+                if (bias) y[v] += bias[j + v];
             }
             float nx[SM][VEC];
 #pragma unroll
@@ -131,7 +133,7 @@ hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __
 
 template <typename TD, typename TO, int S_CT, int VEC>
 static int hc_launch(float* X, const float* x0, const void* delta, int n_partials, size_t ps, const float* mix,
-                     const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, int n_rows, int S,
+                     const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
                      int H, float eps, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
@@ -146,40 +148,40 @@ static int hc_launch(float* X, const float* x0, const void* delta, int n_partial
     int threads = n_rows <= 64 ? 512 : 256;
     while (threads > 64 && threads / 2 >= per) threads /= 2;
     NG_LAUNCH((hc_step_kernel<TD, TO, S_CT, VEC>), n_rows, threads, smem, stream, X, x0, (const TD*)delta, n_partials, ps, mix,
-              out_w, in_w, norm_w, (TO*)out, sum_out, S, H, eps);
+              out_w, in_w, norm_w, (TO*)out, sum_out, bias, S, H, eps);
     return ng_launch_status();
 }
 
 template <typename TD, typename TO>
 static int hc_by_streams(float* X, const float* x0, const void* delta, int n_partials, size_t ps, const float* mix,
-                         const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, int n_rows, int S,
+                         const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
                          int H, float eps, cudaStream_t stream) {
     const bool vec = H % 4 == 0 && ((uintptr_t)X & 15) == 0;
 #define HC_CASE(SS)                                                                                                    \
     case SS:                                                                                                           \
-        return vec ? hc_launch<TD, TO, SS, 4>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream) \
-                   : hc_launch<TD, TO, SS, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream);
+        return vec ? hc_launch<TD, TO, SS, 4>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream) \
+                   : hc_launch<TD, TO, SS, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
     switch (S) {
         HC_CASE(1) HC_CASE(2) HC_CASE(3) HC_CASE(4) HC_CASE(5) HC_CASE(6) HC_CASE(7) HC_CASE(8)
         default:
-            return hc_launch<TD, TO, 0, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream);
+            return hc_launch<TD, TO, 0, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
     }
 }
 
 // delta: null, one [n, H] tensor of the activation type, or (delta_f32) n_partials float32 tensors [n, H] that lie
-// partial_stride elements apart.  x0, in_w (with norm_w and out) and sum_out are optional; mix and out_w go with delta.
+// partial_stride elements apart.  x0, in_w (with norm_w and out), sum_out and bias are optional; mix and out_w go with delta.
 NG_EXPORT int ng_hc_step(float* X, const float* x0, const void* delta, int delta_f32, int n_partials,
                          long long partial_stride, const float* mix, const float* out_w, const float* in_w,
-                         const float* norm_w, void* out, float* sum_out, int n_rows, int S, int H, float eps, int act_bf16,
-                         cudaStream_t stream) {
+                         const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S, int H, float eps,
+                         int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (S < 1 || S > HC_MAX_STREAMS || H <= 0 || n_partials < 1 || (delta && (!mix || !out_w)) || (in_w && (!norm_w || !out)) ||
         (size_t)H * sizeof(float) > 160 * 1024)
         return NG_BAD_SIZE;
     const size_t ps = (size_t)partial_stride;
     if (act_bf16 && delta_f32)
-        return hc_by_streams<float, __nv_bfloat16>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream);
+        return hc_by_streams<float, __nv_bfloat16>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
     if (act_bf16)
-        return hc_by_streams<__nv_bfloat16, __nv_bfloat16>(X, x0, delta, 1, 0, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream);
-    return hc_by_streams<float, float>(X, x0, delta, delta_f32 ? n_partials : 1, ps, mix, out_w, in_w, norm_w, out, sum_out, n_rows, S, H, eps, stream);
+        return hc_by_streams<__nv_bfloat16, __nv_bfloat16>(X, x0, delta, 1, 0, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
+    return hc_by_streams<float, float>(X, x0, delta, delta_f32 ? n_partials : 1, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
 }

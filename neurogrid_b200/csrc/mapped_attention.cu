@@ -13,8 +13,9 @@
 //
 // Two kernels.  ``qkv_prep``: per-head RMS norm of q and k (one weight vector shared by heads and maps; or, `whole`,
 // one norm over all of a row's q and one over all of its k, with weights of that length), q times a temperature
-// 1 + coef * ln(floor((pos + 1) / every) + 1), rotation of the first rot_dims coordinates of every map in pairs (2i, 2i+1), q to its buffer, k and v into
-// their pages.  ``mapped_attention``: a block per (row, query head, run of keys); a warp takes 32 keys of a
+// 1 + coef * ln(floor((pos + 1) / every) + 1), rotation of the first rot_dims coordinates of every map in pairs (2i, 2i+1) or
+// (i, i + rot_dims/2), cosine and sine times `rot_mag`, q to its buffer, k and v into
+// their pages (`v_is_k`: the values are the keys as projected, without norm and rotation).  ``mapped_attention``: a block per (row, query head, run of keys); a warp takes 32 keys of a
 // 128-key tile with a lane per key for the scores of both maps (the key's row read in 16-byte pieces, q from
 // shared memory), keeps an online softmax per map in float32 and adds the weighted values with a lane per pair
 // of value columns; the warps' states are merged in warp order, the runs (few-row steps cut a row's keys into
@@ -35,7 +36,7 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
                 T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ table, int table_stride,
                 const int* __restrict__ positions, const int* __restrict__ row_entry, int nQ, int nK, int nV, int d,
                 int dv, int page_size, int num_pages, float eps, int* __restrict__ status, int whole, float temp_coef,
-                int temp_every, int ld, int half_pairing, int unit_norm) {
+                int temp_every, int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag) {
     extern __shared__ float rot[];                      // cos[rot_dims/2], sin[rot_dims/2]
     __shared__ float red[32];
     ng_pdl_trigger();
@@ -47,8 +48,8 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
     for (int i = threadIdx.x; i < half_rot; i += MA_THREADS) {
         float s, c;
         sincosf((float)pos * inv_freq[i], &s, &c);
-        rot[i] = c;
-        rot[half_rot + i] = s;
+        rot[i] = c * rot_mag;
+        rot[half_rot + i] = s * rot_mag;
     }
     __syncthreads();
     ng_pdl_wait();
@@ -141,7 +142,7 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
         }
     }
     if (page_ok) {
-        const T* vs = in + (size_t)(nQ + nK) * d;
+        const T* vs = in + (size_t)(v_is_k ? nQ : nQ + nK) * d;      // v_is_k: the values are the keys as projected
         for (int j = blockIdx.y * MA_THREADS + threadIdx.x; j < nV * dv; j += MA_THREADS * gridDim.y) {
             const int hv = j / dv, c = j - hv * dv;
             v_pages[v_base + (size_t)hv * page_size * dv + c] = vs[j];
@@ -153,10 +154,13 @@ NG_EXPORT int ng_qkv_prep(const void* qkv, void* q_out, const float* qw, const f
                           int rot_dims, void* k_pages, void* v_pages, const int* table, int table_stride,
                           const int* positions, const int* row_entry, int n_rows, int nQ, int nK, int nV, int d, int dv,
                           int page_size, int num_pages, float eps, int* status, int whole, float temp_coef, int temp_every,
-                          int ld, int half_pairing, int unit_norm, int act_bf16, cudaStream_t stream) {
+                          int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag, int act_bf16,
+                          cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (temp_every < 1 || (whole && (!qw || (nK > 0 && !kw)))) return NG_BAD_SIZE;
-    if (ld < (nQ + nK) * d + nV * dv || (unit_norm && (whole || qw || kw))) return NG_BAD_SIZE;
+    if (ld < (nQ + nK) * d + (v_is_k ? 0 : nV * dv) || (unit_norm && (whole || qw || kw || rot_mag != 1.f)) ||
+        (v_is_k && (nV != nK || dv != d)))
+        return NG_BAD_SIZE;
     if (d <= 0 || d > 64 * MA_MAX_PAIRS || dv <= 0 || nQ <= 0 || nK < 0 || nV < 0 || page_size <= 0 || rot_dims < 0 ||
         rot_dims > d || (rot_dims & 1) || (rot_dims > 0 && !inv_freq))
         return NG_BAD_SIZE;
@@ -167,11 +171,11 @@ NG_EXPORT int ng_qkv_prep(const void* qkv, void* q_out, const float* qw, const f
         NG_LAUNCH((qkv_prep_kernel<__nv_bfloat16>), grid, MA_THREADS, smem, stream, (const __nv_bfloat16*)qkv,
                   (__nv_bfloat16*)q_out, qw, kw, inv_freq, rot_dims, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, table,
                   table_stride, positions, row_entry, nQ, nK, nV, d, dv, page_size, num_pages, eps, status, whole, temp_coef,
-                  temp_every, ld, half_pairing, unit_norm);
+                  temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag);
     else
         NG_LAUNCH((qkv_prep_kernel<float>), grid, MA_THREADS, smem, stream, (const float*)qkv, (float*)q_out, qw, kw,
                   inv_freq, rot_dims, (float*)k_pages, (float*)v_pages, table, table_stride, positions, row_entry, nQ, nK, nV,
-                  d, dv, page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm);
+                  d, dv, page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag);
     return ng_launch_status();
 }
 

@@ -106,6 +106,19 @@ def embed(table: torch.Tensor, tokens: torch.Tensor, out: torch.Tensor, status: 
              n, H, V, _ptr(status), int(accumulate), 4 if accumulate else 1, float(scale), _stream()), "embed")
 
 
+def embed_norm(table: torch.Tensor, tokens: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, status: torch.Tensor,
+               eps: float, scale: float = 1.0) -> None:
+    """out[N,H] (float32) = rmsnorm(table[tokens] * scale) * weight; a token outside the table gives zeros and a status bit."""
+    n, H = out.shape
+    if table.shape[1] != H or weight.numel() != H or tokens.numel() != n:
+        raise KernelError("embed_norm: shapes do not fit")
+    _f32(out, "embed out"), _f32(weight, "norm weight"), _i32(tokens, "tokens"), _i32(status, "status")
+    f = _fn("elementwise", "ng_embed_norm", [_c_void_p, _c_int] + [_c_void_p] * 3 + [_c_int] * 3 + [_c_void_p, _c_float, _c_float,
+                                                                                                _c_void_p])
+    _check(f(_ptr(table, "embedding table"), _act_flag(table, "embedding table"), _ptr(tokens), _ptr(weight), _ptr(out), n, H,
+             table.shape[0], _ptr(status), float(scale), float(eps), _stream()), "embed_norm")
+
+
 def _partials(delta: Optional[torch.Tensor], h: torch.Tensor, act: int):
     """(delta_f32, n_partials, stride): ``delta`` is [N,H] of the activation dtype, or a stack
     [S,N,H] of float32 partial sums (split-K products) that are added in ascending order."""
@@ -164,7 +177,7 @@ def residual_add(h: torch.Tensor, delta: torch.Tensor) -> None:
     _check(f(_ptr(h), _ptr(delta), h.numel(), int(delta.dtype == torch.bfloat16), n_part, _stream()), "residual_add")
 
 
-GATE_ACTIVATIONS = ("silu", "gelu_tanh")
+GATE_ACTIVATIONS = ("silu", "gelu_tanh", "clamped_glu")
 
 
 def _column_block(out: torch.Tensor, what: str) -> int:
@@ -174,16 +187,17 @@ def _column_block(out: torch.Tensor, what: str) -> int:
     return out.stride(0) if out.shape[0] > 1 else max(out.stride(0), out.shape[1])
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out[N,I] = act(gate_up[:, :I]) * gate_up[:, I:], act = silu or the tanh form of gelu.  ``out`` may be a block
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu", limit: float = 0.0, alpha: float = 0.0) -> None:
+    """out[N,I] = act(gate_up[:, :I]) * gate_up[:, I:], act = silu or the tanh form of gelu; "clamped_glu":
+    g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit).  ``out`` may be a block
     of columns of a wider buffer."""
     n, I = out.shape
     if gate_up.shape != (n, 2 * I) or gate_up.dtype != out.dtype or activation not in GATE_ACTIVATIONS:
         raise KernelError(f"swiglu: gate_up {tuple(gate_up.shape)} does not match out {tuple(out.shape)}")
     ldo = _column_block(out, "swiglu out")
-    f = _fn("elementwise", "ng_swiglu", [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p])
-    _check(f(_ptr(gate_up), out.data_ptr(), n, I, ldo, int(activation == "gelu_tanh"), _act_flag(out, "swiglu out"),
-             _stream()), "swiglu")
+    f = _fn("elementwise", "ng_swiglu", [_c_void_p, _c_void_p] + [_c_int] * 4 + [_c_float, _c_float, _c_int, _c_void_p])
+    _check(f(_ptr(gate_up), out.data_ptr(), n, I, ldo, GATE_ACTIVATIONS.index(activation), float(limit), float(alpha),
+             _act_flag(out, "swiglu out"), _stream()), "swiglu")
 
 
 # ----------------------------------------------------------------------------- float32 product
@@ -391,7 +405,8 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
              inv_freq: Optional[torch.Tensor], k_pages: Optional[torch.Tensor], v_pages: Optional[torch.Tensor],
              table: torch.Tensor, positions: torch.Tensor, row_entry: torch.Tensor, n_q: int, n_k: int, n_v: int,
              dim: int, vdim: int, eps: float, status: torch.Tensor, *, whole: bool = False, q_temp_coef: float = 0.0,
-             q_temp_every: int = 1, half_pairing: bool = False, unit_norm: bool = False) -> None:
+             q_temp_every: int = 1, half_pairing: bool = False, unit_norm: bool = False, v_is_k: bool = False,
+             rot_mag: float = 1.0) -> None:
     """qkv[N, (n_q + n_k) * dim + n_v * vdim]: every q and k head (a map of a head counts as one) gets its RMS norm
     over ``dim`` (if its weight is given; float32, shared by all heads) and the rotation of its first
     2 * len(inv_freq) coordinates in pairs (2i, 2i+1) by position * inv_freq[i]; q -> q_out[N, n_q * dim],
@@ -400,10 +415,13 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
     all of its k, the weights then float32 [n_q * dim] and [n_k * dim].  ``q_temp_coef`` c, ``q_temp_every`` m: q is
     multiplied by 1 + c * ln(floor((position + 1) / m) + 1) after its norm.  ``half_pairing``: the rotated coordinates
     pair as (i, i + rot_dims/2).  ``unit_norm`` (without norm weights): every q and k head is divided by its root mean
-    square all the same.  ``qkv`` may have further columns behind v; they are not read."""
+    square all the same.  ``qkv`` may have further columns behind v; they are not read.  ``v_is_k``: there are no v columns,
+    the values are the keys as projected (no norm, no rotation; n_v = n_k, vdim = dim).  ``rot_mag`` multiplies cosines
+    and sines."""
     n = q_out.shape[0]
     if q_out.shape != (n, n_q * dim) or qkv.dim() != 2 or qkv.shape[0] != n \
-            or qkv.shape[1] < (n_q + n_k) * dim + n_v * vdim or qkv.dtype != q_out.dtype:
+            or qkv.shape[1] < (n_q + n_k) * dim + (0 if v_is_k else n_v * vdim) or qkv.dtype != q_out.dtype \
+            or (v_is_k and (n_v != n_k or vdim != dim)):
         raise KernelError("qkv_prep: shapes or dtypes do not fit")
     page_size = num_pages = 1
     if n_k or n_v:
@@ -417,12 +435,13 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
     if whole and (q_weight is None or q_weight.numel() != n_q * dim or (n_k and (k_weight is None or k_weight.numel() != n_k * dim))):
         raise KernelError("qkv_prep: a norm over the whole projection needs weights of the projection's length")
     f = _fn("mapped_attention", "ng_qkv_prep", [_c_void_p] * 5 + [_c_int] + [_c_void_p] * 3 + [_c_int] + [_c_void_p] * 2
-            + [_c_int] * 8 + [_c_float, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p])
+            + [_c_int] * 8 + [_c_float, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int,
+                              _c_void_p])
     _check(f(_ptr(qkv), _ptr(q_out), _ptr(q_weight), _ptr(k_weight), _ptr(inv_freq), rot_dims,
              _ptr(k_pages) if n_k else None, _ptr(v_pages) if n_v else None, _ptr(table), table.shape[1], _ptr(positions),
              _ptr(row_entry), n, n_q, n_k, n_v, dim, vdim, page_size, num_pages, float(eps), _ptr(status),
              int(bool(whole)), float(q_temp_coef), int(q_temp_every), qkv.shape[1], int(bool(half_pairing)),
-             int(bool(unit_norm)), _act_flag(q_out, "q_out"), _stream()), "qkv_prep")
+             int(bool(unit_norm)), int(bool(v_is_k)), float(rot_mag), _act_flag(q_out, "q_out"), _stream()), "qkv_prep")
 
 
 def mapped_attention_partial_floats(n_rows: int, n_heads: int, n_maps: int, vdim: int, n_splits: int) -> int:
@@ -872,18 +891,20 @@ def gate_mul(y: torch.Tensor, gate: Optional[torch.Tensor], activation: str = "s
 def hc_step(streams: torch.Tensor, n_streams: int, *, x0: Optional[torch.Tensor] = None, delta: Optional[torch.Tensor] = None,
             mix: Optional[torch.Tensor] = None, out_w: Optional[torch.Tensor] = None, in_w: Optional[torch.Tensor] = None,
             norm_w: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-            sum_out: Optional[torch.Tensor] = None, eps: float = 0.0, act_dtype=None) -> None:
+            sum_out: Optional[torch.Tensor] = None, eps: float = 0.0, act_dtype=None, bias: Optional[torch.Tensor] = None) -> None:
     """What lies between two sublayers of a model whose residual stream is ``n_streams`` copies, streams[N, S * H]
     float32.  ``x0`` [N,H] float32: every copy is x0 (a sequence's start).  ``delta`` (the output y of the sublayer
     before: [N,H] of the activation dtype or a float32 stack of partial sums) with ``mix`` [S,S] ([from, to]) and
-    ``out_w`` [S]: x_t <- sum_s mix[s,t] x_s + out_w[t] y for all t at once.  ``in_w`` [S] with ``norm_w`` [H] and
+    ``out_w`` [S]: x_t <- sum_s mix[s,t] x_s + out_w[t] y for all t at once (``bias`` [H] float32 belongs to y: it is added to it).  ``in_w`` [S] with ``norm_w`` [H] and
     ``out`` [N,H]: out = rmsnorm(sum_t in_w[t] x_t) * norm_w.  ``sum_out`` [N,H] float32: the sum of the copies."""
     n = streams.shape[0]
     H = streams.shape[1] // n_streams
     if streams.shape[1] != n_streams * H:
         raise KernelError("hc_step: the streams do not divide into copies")
     _f32(streams, "streams"), _f32(x0, "x0"), _f32(mix, "mix"), _f32(out_w, "out_w"), _f32(in_w, "in_w"), _f32(norm_w, "norm weight")
-    _f32(sum_out, "sum_out")
+    _f32(sum_out, "sum_out"), _f32(bias, "bias")
+    if bias is not None and bias.numel() != H:
+        raise KernelError("hc_step: the bias is [H]")
     act_dtype = out.dtype if out is not None else (act_dtype or torch.float32)
     act = int(act_dtype == torch.bfloat16)
     d32, n_part, stride = 0, 1, 0
@@ -896,10 +917,10 @@ def hc_step(streams: torch.Tensor, n_streams: int, *, x0: Optional[torch.Tensor]
     for t in (x0, sum_out):
         if t is not None and t.shape != (n, H):
             raise KernelError("hc_step: x0 and sum_out are [N, H]")
-    f = _fn("hyper", "ng_hc_step", [_c_void_p] * 3 + [_c_int, _c_int, _c_ll] + [_c_void_p] * 6 + [_c_int] * 3
+    f = _fn("hyper", "ng_hc_step", [_c_void_p] * 3 + [_c_int, _c_int, _c_ll] + [_c_void_p] * 7 + [_c_int] * 3
             + [_c_float, _c_int, _c_void_p])
     _check(f(_ptr(streams), _ptr(x0), _ptr(delta), d32, n_part, stride, _ptr(mix), _ptr(out_w), _ptr(in_w), _ptr(norm_w),
-             _ptr(out), _ptr(sum_out), n, int(n_streams), H, float(eps), act, _stream()), "hc_step")
+             _ptr(out), _ptr(sum_out), _ptr(bias), n, int(n_streams), H, float(eps), act, _stream()), "hc_step")
 
 
 # ----------------------------------------------------------------------------- gated linear attention
@@ -949,6 +970,90 @@ def gated_linear_chunked_takes(key_dim: int, value_dim: int) -> bool:
     """Whether the chunk-by-chunk kernels take the head sizes."""
     f = _fn("gated_linear", "ng_gated_linear_chunked_takes", [_c_int, _c_int])
     return bool(f(int(key_dim), int(value_dim)))
+
+
+# ----------------------------------------------------------------------------- linear attention with a scalar decay
+DECAYED_CHUNK = 64           # tokens of a chunk in the chunk-by-chunk kernels
+
+
+def decayed_linear_slices(value_dim: int) -> int:
+    """Copies of a head's normaliser and running maximum that the token-by-token kernel's blocks keep."""
+    return -(-value_dim // 32)
+
+
+def decayed_linear_chunked_takes(key_dim: int, value_dim: int) -> bool:
+    """Whether the chunk-by-chunk tensor-core kernels take the head sizes."""
+    return key_dim % 16 == 0 and value_dim % 16 == 0 and 16 <= key_dim <= 256 and value_dim >= 16
+
+
+def decayed_linear_scratch(n_rows: int, n_entries: int, n_heads: int, key_dim: int, value_dim: int) -> int:
+    """float32 values the chunk-by-chunk kernels need: per chunk and head the state and normaliser before it, per token
+    and head its gates."""
+    slots = n_rows // DECAYED_CHUNK + n_entries + 1
+    return slots * n_heads * (key_dim * value_dim + key_dim + 2) + n_rows * n_heads * 4 + 8
+
+
+def _decayed_linear(what, x, gates, gate_bias, decay, cap, state, nm_state, o_raw, norm_w, out, cu_q, ctx_before, slots,
+                    row_entry, n_entries, n_heads, key_dim, value_dim, norm_group, eps, out_scale, scratch, max_q):
+    n = x.shape[0]
+    width = n_heads * value_dim
+    if x.shape[1] != 2 * n_heads * (key_dim + value_dim) or out.shape != (n, width) or out.dtype != x.dtype \
+            or o_raw.shape != (n, width) or norm_w.numel() != width or state.shape[1:] != (n_heads, key_dim, value_dim):
+        raise KernelError(f"{what}: shapes or dtypes do not fit")
+    for t, w in ((state, "state"), (nm_state, "normaliser state"), (o_raw, "output scratch"), (norm_w, "norm weight"),
+                 (gates, "gates"), (gate_bias, "gate biases"), (decay, "decay"), (scratch, "scratch")):
+        _f32(t, w)
+    _i32(cu_q, "cu_q"), _i32(ctx_before, "ctx_before"), _i32(slots, "slots"), _i32(row_entry, "row_entry")
+    act = _act_flag(x, f"{what} input")
+    common = (_ptr(x), _ptr(gates), _ptr(gate_bias), _ptr(decay), float(cap), _ptr(state), _ptr(nm_state), _ptr(o_raw))
+    if scratch is not None:
+        need = decayed_linear_scratch(n, n_entries, n_heads, key_dim, value_dim)
+        if scratch.numel() < need or max_q <= 0 or x.dtype != torch.bfloat16 or not decayed_linear_chunked_takes(key_dim, value_dim):
+            raise KernelError(f"{what}: the chunked kernels take bfloat16 and heads in sixteens, and need {need} float32 values "
+                              "of scratch and the longest portion's length")
+        f = _fn("decayed_linear", "ng_dl_chunked", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 7 + [_c_int] * 6 + [_c_void_p])
+        _check(f(*common, _ptr(scratch), _ptr(cu_q), _ptr(ctx_before), _ptr(slots), n_entries, n, int(max_q), n_heads, key_dim,
+                 value_dim, _stream()), f"{what} (chunked)")
+    else:
+        f = _fn("decayed_linear", "ng_dl_step", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 6 + [_c_int] * 5 + [_c_void_p])
+        _check(f(*common, _ptr(cu_q), _ptr(ctx_before), _ptr(slots), n_entries, n_heads, key_dim, value_dim, act, _stream()), what)
+    gate_at = 2 * n_heads * key_dim + width                     # the output gate's columns of x
+    f = _fn("decayed_linear", "ng_dl_finish", [_c_void_p] * 5 + [_c_int] * 5 + [_c_float, _c_float, _c_int, _c_void_p])
+    _check(f(_ptr(o_raw), x.data_ptr() + gate_at * x.element_size(), _ptr(norm_w), out.data_ptr(), _ptr(row_entry), n, width,
+             int(norm_group), x.shape[1], _column_block(out, f"{what} out"), float(eps), float(out_scale), act, _stream()),
+           f"{what} (norm and gate)")
+
+
+def lightning(x: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state: torch.Tensor, o_raw: torch.Tensor,
+              out: torch.Tensor, cu_q: torch.Tensor, ctx_before: torch.Tensor, slots: torch.Tensor, row_entry: torch.Tensor,
+              n_entries: int, n_heads: int, key_dim: int, value_dim: int, eps: float, out_scale: float = 1.0,
+              scratch: Optional[torch.Tensor] = None, max_q: int = 0) -> None:
+    """x[N, 2*nH*(dk+dv)] = q|k|v|g;  q, k, v <- silu (rounded to x's dtype);  per head S = decay*S + k v^T, o = S^T q;
+    out[N, nH*dv] = o / rms(o over all heads together) * norm_w * sigmoid(g) * out_scale;  state[slots, nH, dk, dv] and
+    the scratch ``o_raw`` [N, nH*dv] float32.  ``out`` may be a block of columns of a wider buffer.  With ``scratch``
+    (``decayed_linear_scratch`` float32 values) and ``max_q`` (the longest portion) the chunk-by-chunk tensor-core
+    kernels run (bfloat16; ``decayed_linear_chunked_takes``); else the token-by-token kernel."""
+    if decay.numel() != n_heads:
+        raise KernelError("lightning: a decay per head")
+    _decayed_linear("lightning", x, None, None, decay, 0.0, state, None, o_raw, norm_w, out, cu_q, ctx_before, slots, row_entry,
+                    n_entries, n_heads, key_dim, value_dim, n_heads * value_dim, eps, out_scale, scratch, max_q)
+
+
+def mlstm(x: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: float, norm_w: torch.Tensor,
+          state: torch.Tensor, nm_state: torch.Tensor, o_raw: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor,
+          ctx_before: torch.Tensor, slots: torch.Tensor, row_entry: torch.Tensor, n_entries: int, n_heads: int, key_dim: int,
+          value_dim: int, eps: float, out_scale: float = 1.0, scratch: Optional[torch.Tensor] = None, max_q: int = 0) -> None:
+    """x[N, 2*nH*(dk+dv)] = q|k|v|g and gates[N, 2*nH] float32 = preactivations i|f (``gate_bias`` [2*nH] is added here):
+    i = cap tanh(./cap), f = log sigmoid(cap tanh(./cap)), m' = max(f + m, i), S = exp(f + m - m') S + exp(i - m') k v^T,
+    n likewise with k alone, o = s S^T q / (max(|s n.q|, exp(-m')) + 1e-6), s = dk^(-1/2);
+    out[N, nH*dv] = o / rms(o of the head) * norm_w * sigmoid(g) * out_scale.  state[slots, nH, dk, dv] and
+    nm_state[slots, nH, ``decayed_linear_slices(dv)``, dk+1] (n | m, one copy per slice) float32.  The rest as ``lightning``."""
+    n = x.shape[0]
+    if gates.shape != (n, 2 * n_heads) or gate_bias.numel() != 2 * n_heads \
+            or nm_state.shape[1:] != (n_heads, decayed_linear_slices(value_dim), key_dim + 1):
+        raise KernelError("mlstm: shapes do not fit")
+    _decayed_linear("mlstm", x, gates, gate_bias, None, cap, state, nm_state, o_raw, norm_w, out, cu_q, ctx_before, slots,
+                    row_entry, n_entries, n_heads, key_dim, value_dim, value_dim, eps, out_scale, scratch, max_q)
 
 
 def scale_(x: torch.Tensor, factor: float) -> None:
@@ -1078,7 +1183,7 @@ def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor], top_p: Opt
 
 
 # ----------------------------------------------------------------------------- tensor-core products
-_GEMM_ARGS = [_c_void_p] * 4 + [_c_int] * 9 + [_c_void_p, _c_void_p]
+_GEMM_ARGS = [_c_void_p] * 4 + [_c_int] * 9 + [_c_float, _c_float, _c_void_p, _c_void_p]
 # Steps of at most FUSE_MAX_ROWS rows (bfloat16, tcgen05 backend) add the products that end a
 # mixer or a feed-forward straight into the float32 residual stream (red.global.add in the
 # epilogue): the norm kernel that follows has no partial sums to read.  Measured on the decode
@@ -1142,7 +1247,7 @@ def gemm_sm100(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], o
         if bias is not None or tuple(out.shape) not in (((M, N),) if s_eff == 1 else ()) + ((s_eff, M, N),):
             raise KernelError(f"gemm_sm100: float32 output must be [{s_eff}, {M}, {N}] (no bias)")
     f = _fn("gemm_sm100", "ng_gemm_sm100", _GEMM_ARGS)
-    _check(f(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), M, N, K, N, N, epi, s_eff, 0, token_tile,
+    _check(f(_ptr(x), _ptr(w), _ptr(bias), _ptr(out), M, N, K, N, N, epi, s_eff, 0, token_tile, 0.0, 0.0,
              _ptr(_gemm_status(x.device)), _stream()), "gemm_sm100")
 
 
@@ -1154,9 +1259,9 @@ def gemm_splits(K: int, splits: int) -> int:
 
 
 def gemm_swiglu_sm100(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, *, token_tile: int = 0,
-                      activation: str = "silu") -> None:
+                      activation: str = "silu", limit: float = 0.0, alpha: float = 0.0) -> None:
     """out[M,I] = act(x wg^T) * (x wu^T) with w_gate_up = [wg (I rows); wu (I rows)]: the gate is
-    applied in the product's epilogue (act = silu or the tanh form of gelu).  ``out`` may be a block of columns
+    applied in the product's epilogue (act = silu or the tanh form of gelu, or both halves clamped, as ``swiglu`` has them).  ``out`` may be a block of columns
     of a wider buffer."""
     M, K = x.shape
     I = out.shape[1]
@@ -1165,8 +1270,8 @@ def gemm_swiglu_sm100(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tenso
     ldc = _column_block(out, "gemm_swiglu_sm100 out")
     status = _ptr(_gemm_status(w_gate_up.device))
     f = _fn("gemm_sm100", "ng_gemm_sm100", _GEMM_ARGS)
-    _check(f(_ptr(x), _ptr(w_gate_up), None, out.data_ptr(), M, I, K, 2 * I, ldc, 4 if activation == "gelu_tanh" else 2, 1, I,
-             token_tile, status, _stream()), "gemm_swiglu_sm100")
+    _check(f(_ptr(x), _ptr(w_gate_up), None, out.data_ptr(), M, I, K, 2 * I, ldc,
+             {"silu": 2, "gelu_tanh": 4, "clamped_glu": 6}[activation], 1, I, token_tile, float(limit), float(alpha), status, _stream()), "gemm_swiglu_sm100")
 
 
 # ----------------------------------------------------------------------------- matrix products
@@ -1201,7 +1306,7 @@ def linear_to_residual(x: torch.Tensor, weight: torch.Tensor, bias: Optional[tor
         if FUSE_RED and residual is not None and M <= FUSE_MAX_ROWS:
             _f32(residual, "residual")
             f = _fn("gemm_sm100", "ng_gemm_sm100", _GEMM_ARGS)
-            _check(f(_ptr(x), _ptr(weight), None, _ptr(residual), M, N, K, N, N, 3, s, 0, 0,
+            _check(f(_ptr(x), _ptr(weight), None, _ptr(residual), M, N, K, N, N, 3, s, 0, 0, 0.0, 0.0,
                      _ptr(_gemm_status(weight.device)), _stream()), "gemm_sm100 (residual add)")
             return None
         if s > 1:

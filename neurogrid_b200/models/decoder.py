@@ -37,6 +37,7 @@ class Decoder:
         self.head_weight: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None
         self.pair_table: Optional[torch.Tensor] = None
+        self.embed_norm = registry.build("norm", spec.embed_norm, dtype=dtype, device=device) if spec.embed_norm is not None else None
 
     # ------------------------------------------------------------------ weights
     def tensors(self) -> Dict[str, TensorDecl]:
@@ -49,6 +50,9 @@ class Decoder:
             out.update(getattr(block, "shared_tensors", dict)())
         for name, decl in self.final_norm.tensors().items():
             out[_join(s.final_norm_name, name)] = decl
+        if self.embed_norm is not None:
+            for name, decl in self.embed_norm.tensors().items():
+                out[_join(s.embed_norm_name, name)] = decl
         if not s.tie_head:
             out[s.head_name] = TensorDecl((s.vocab_size, s.hidden))
         if s.position_table_name:
@@ -70,6 +74,8 @@ class Decoder:
             if hasattr(block, "bind_shared"):
                 block.bind_shared(weights)
         self.final_norm.bind({rel: weights[_join(s.final_norm_name, rel)] for rel in self.final_norm.tensors()})
+        if self.embed_norm is not None:
+            self.embed_norm.bind({rel: weights[_join(s.embed_norm_name, rel)] for rel in self.embed_norm.tensors()})
 
     def cache_needs(self) -> Dict[int, object]:
         """Cache id -> what the layers that use it need to keep between steps."""
@@ -150,7 +156,11 @@ class Decoder:
         own, from which the first block's first kernel makes every copy."""
         s = self.spec
         h = ctx.ws.buf("embedded" if s.streams else "residual", ctx.n_rows, s.hidden, torch.float32)
-        ops.embed(self.embed_table, ctx.tokens, h, ctx.status, scale=s.embed_scale)
+        if self.embed_norm is not None:                      # one kernel for the embedding and its norm
+            ops.embed_norm(self.embed_table, ctx.tokens, self.embed_norm.weight, h, ctx.status, self.embed_norm.spec.eps,
+                           scale=s.embed_scale)
+        else:
+            ops.embed(self.embed_table, ctx.tokens, h, ctx.status, scale=s.embed_scale)
         if self.position_table is not None:                  # learned absolute positions: h += table[position]
             ops.embed(self.position_table, ctx.positions, h, ctx.status, accumulate=True)
         if self.pair_table is not None:                      # the pair (previous token, token): h += table[row of the pair]
@@ -185,8 +195,8 @@ class Decoder:
         elif pending is None:
             ops.hc_step(h, s.streams, sum_out=total, act_dtype=self.dtype)
         else:
-            ops.hc_step(h, s.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, sum_out=total,
-                        act_dtype=self.dtype)
+            ops.hc_step(h, s.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, bias=pending.bias,
+                        sum_out=total, act_dtype=self.dtype)
         return total
 
     def finish(self, ctx: StepContext, h: torch.Tensor, pending, want_rows: Optional[torch.Tensor],

@@ -96,6 +96,7 @@ class PositionArgs:
     pos_scale: float = 1.0
     score_slopes: Optional[torch.Tensor] = None
     rotary_dims: Optional[int] = None      # a partial rotation: only the first that many coordinates of a head
+    magnitude: float = 1.0                 # cosines and sines are multiplied by this
 
     @classmethod
     def of(cls, args) -> "PositionArgs":

@@ -254,10 +254,11 @@ class ParallelBlock:
 
 class HyperPending:
     """What a hyper block leaves for the kernel after it: its last sublayer's output (not yet written into the copies of
-    the stream) with the mixing matrix and output weights that write it."""
+    the stream; ``bias``, float32 [H] or None, is still to be added to it) with the mixing matrix and output weights that
+    write it."""
 
-    def __init__(self, y, mix, out_w, eps):
-        self.y, self.mix, self.out_w, self.eps = y, mix, out_w, eps
+    def __init__(self, y, mix, out_w, eps, bias=None):
+        self.y, self.mix, self.out_w, self.eps, self.bias = y, mix, out_w, eps, bias
 
 
 @register("block", "hyper")
@@ -265,7 +266,10 @@ class HyperBlock:
     """Pre-norm with hyper-connections: the residual stream is S copies x_1..x_S (``spec.options["streams"]``).  For
     sublayer q (the mixer, then the feed-forward if there is one), with vectors in_q, out_q [S] and a matrix mix_q [S,S]:
 
-        u = sum_s in_q[s] x_s;   y = sublayer(norm_q(u));   x_t <- sum_s mix_q[s, t] x_s + out_q[t] y   (all t at once)
+        u = sum_s in_q[s] x_s;   y = sublayer(norm_q(u));   x_t <- sum_s mix_q[s, t] x_s + r out_q[t] y   (all t at once)
+
+    with r = ``spec.options["residual_mult"]`` (1 if not given; multiplied into out_q when bound, float32).
+    ``spec.options["plain"]``: one copy and no tensors, in = mix = 1 and out = r: the ordinary residual sum x + r y.
 
     The copies are float32 [N, S * H] (the buffer the model hands over as its stream).  One kernel does what lies
     between two sublayers: the update by the sublayer before (also the last one of the layer before, handed over as
@@ -277,6 +281,10 @@ class HyperBlock:
     def __init__(self, spec, *, dtype, device, owns_cache=True):
         self.spec, self.dtype, self.device = spec, dtype, device
         self.streams = int(spec.options["streams"])
+        self.mult = float(spec.options.get("residual_mult", 1.0))
+        self.plain = bool(spec.options.get("plain", False))
+        if self.plain and self.streams != 1:
+            raise ValueError("plain residual sums have one copy of the stream")
         kw = dict(dtype=dtype, device=device)
         mixer_kw = dict(kw)
         if not owns_cache:
@@ -286,6 +294,8 @@ class HyperBlock:
         self.mixer_norm = registry.build("norm", spec.mixer_norm, **kw)
         self.ffn_norm = registry.build("norm", spec.ffn_norm, **kw) if spec.ffn is not None else None
         self.hc = {}
+        if hasattr(self.mixer, "defer_bias"):                # its output's bias rides in the kernel behind it
+            self.mixer.defer_bias = True
 
     def parts(self):
         n = self.spec.names
@@ -302,7 +312,7 @@ class HyperBlock:
         for sub, part in self.parts().items():
             for name, decl in part.tensors().items():
                 out[f"{sub}.{name}" if name else sub] = decl
-        for hc in self._hc_names():
+        for hc in self._hc_names() if not self.plain else ():
             out[hc + ".in"] = TensorDecl((S,), "share")
             out[hc + ".out"] = TensorDecl((S,), "norm")
             out[hc + ".mix"] = TensorDecl((S, S), "eye")
@@ -318,7 +328,9 @@ class HyperBlock:
             part.bind(own)
         f32 = dict(device=self.device, dtype=torch.float32)
         for hc in self._hc_names():
-            self.hc[hc] = tuple(t[f"{hc}.{k}"].to(**f32).contiguous() for k in ("in", "out", "mix"))
+            w_in, w_out, mix = (torch.ones(1, **f32) if self.plain else t[f"{hc}.{k}"].to(**f32).contiguous()
+                                for k in ("in", "out", "mix"))
+            self.hc[hc] = (w_in, w_out if self.mult == 1.0 else (w_out * self.mult).contiguous(), mix)
 
     def cache_need(self):
         return self.mixer.cache_need()
@@ -340,7 +352,7 @@ class HyperBlock:
         elif pending is None:
             ops.hc_step(X, self.streams, **kw)
         else:
-            ops.hc_step(X, self.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, **kw)
+            ops.hc_step(X, self.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, bias=pending.bias, **kw)
         return buf
 
     def forward(self, X, pending, ctx, cache):
@@ -351,7 +363,8 @@ class HyperBlock:
         names = self._hc_names()
         x = self._between(X, pending, names[0], self.mixer_norm, buf)
         y = self.mixer.forward(x, ctx, cache)
-        pending = HyperPending(y, self.hc[names[0]][2], self.hc[names[0]][1], self.spec.mixer_norm.eps)
+        pending = HyperPending(y, self.hc[names[0]][2], self.hc[names[0]][1], self.spec.mixer_norm.eps,
+                               bias=self.mixer.out_bias if getattr(self.mixer, "defer_bias", False) else None)
         if self.ffn is not None:
             x = self._between(X, pending, names[1], self.ffn_norm, buf)
             y = self.ffn.forward(x, ctx)

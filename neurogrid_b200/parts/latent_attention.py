@@ -94,6 +94,8 @@ class LatentAttention:
         the encoding's rotated coordinates get the frequency zero (they pass unchanged)."""
         if getattr(self, "_pa", None) is None:
             pa = PositionArgs.of(self.position.kernel_args())
+            if pa.magnitude != 1.0:
+                raise NotImplementedError("the rotated part takes rotations that keep lengths")
             if pa.pos_scale != 1.0 or (pa.half_pairing and pa.inv_freq is not None and pa.inv_freq.numel() != self.rope // 2):
                 raise NotImplementedError("the rotated part takes unscaled positions, and pairs (i, i + half) only whole")
             f = torch.zeros(self.rope // 2, dtype=torch.float32, device=self.device)

@@ -39,16 +39,18 @@ class MappedAttention:
         self.spec, self.dtype, self.device, self.owns_cache = spec, dtype, device, owns_cache
         self.position = registry.build("position", spec.position, device=device)
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_norm = self.k_norm = self.sinks = None
+        self.b_o_f32 = None           # the output projection's bias as stored
         self.lam = 0.0
+        self.shared_kv = getattr(spec, "shared_kv", False)                    # the values are the keys as projected
         self.whole = getattr(spec, "norm_scope", "head") == "projection"      # one norm over all of q, one over all of k
 
     def _proj(self):
-        """The stacked projection's parts in order: q, k, v (a layer that reads another's cache: q only), then the
-        output gate's logits if the mixer has one."""
+        """The stacked projection's parts in order: q, k, v (a layer that reads another's cache: q only; one whose values
+        are its keys: no v), then the output gate's logits if the mixer has one."""
         s = self.spec
         rows = {"q": s.n_heads * s.n_maps * s.key_dim, "k": s.n_kv_heads * s.n_maps * s.key_dim,
                 "v": s.n_kv_heads * s.value_dim, "out_gate": s.n_heads * s.value_dim}
-        parts = ("q", "k", "v") if self.owns_cache else ("q",)
+        parts = (("q", "k") if self.shared_kv else ("q", "k", "v")) if self.owns_cache else ("q",)
         return {p: rows[p] for p in parts + (("out_gate",) if getattr(s, "out_gate", False) else ())}
 
     def tensors(self):
@@ -80,12 +82,15 @@ class MappedAttention:
         if s.bias:
             self.b_qkv = torch.cat([t[n[p + "_bias"]].to(**kw) for p in self._proj()]).contiguous()
             self.b_o = t[n["o_bias"]].to(**kw).contiguous()
+            self.b_o_f32 = t[n["o_bias"]].to(**f32).contiguous()
         if s.qk_norm and getattr(s, "norm_weight", True):
             self.q_norm = t[n["q_norm"]].to(**f32).contiguous()
             if self.owns_cache:
                 self.k_norm = t[n["k_norm"]].to(**f32).contiguous()
         if getattr(s, "sink", False):
             self.sinks = t[n["sink"]].to(**f32).contiguous()
+        elif getattr(s, "unit_sink", False):
+            self.sinks = torch.zeros(s.n_heads, **f32)
         if s.n_maps == 2:            # one number per layer, formed in float32 as the stored vectors' products
             v = {k: t[n[k]].to(torch.float32) for k in ("lq1", "lk1", "lq2", "lk2")}
             self.lam = float(torch.exp((v["lq1"] * v["lk1"]).sum()) - torch.exp((v["lq2"] * v["lk2"]).sum())) + float(s.diff)
@@ -166,7 +171,8 @@ class MappedAttention:
                      s.key_dim, s.value_dim, s.eps, ctx.status, whole=self.whole,
                      q_temp_coef=getattr(s, "q_temp_coef", 0.0), q_temp_every=getattr(s, "q_temp_every", 1),
                      half_pairing=bool(pa.inv_freq is not None and pa.half_pairing),
-                     unit_norm=bool(s.qk_norm and not getattr(s, "norm_weight", True)))
+                     unit_norm=bool(s.qk_norm and not getattr(s, "norm_weight", True)),
+                     v_is_k=bool(self.shared_kv and n_v), rot_mag=pa.magnitude if pa.inv_freq is not None else 1.0)
         self.attend(q, cache, ctx, out, pa.score_slopes)
         if gated or out_scale != 1.0:
             ops.gate_mul(out, gate, "sigmoid", out_scale)

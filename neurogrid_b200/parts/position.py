@@ -29,11 +29,19 @@ class Rope:
             s = (original / wavelength - low) / (high - low) if high != low else torch.ones_like(f)
             blend = (1.0 - s) * f / factor + s * f
             f = torch.where(wavelength < original / high, f, torch.where(wavelength > original / low, f / factor, blend))
+        self.magnitude = 1.0
+        if spec.yarn is not None:                          # by index: pairs that turn too seldom within `original` positions are divided
+            factor, original, fast, slow = (float(v) for v in spec.yarn)
+            at = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(float(spec.theta)))
+            lo, hi = max(math.floor(at(fast)), 0), min(math.ceil(at(slow)), dims - 1)
+            ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
+            f = f / factor * ramp + f * (1.0 - ramp)
+            self.magnitude = 0.1 * math.log(factor) + 1.0
         self.inv_freq = f.to(torch.float32).to(device)
 
     def kernel_args(self):
         return PositionArgs(self.inv_freq, self.spec.pairing == "half", float(self.spec.scale),
-                            rotary_dims=self.spec.rotary_dims)
+                            rotary_dims=self.spec.rotary_dims, magnitude=self.magnitude)
 
 
 @register("position", "distance_bias")

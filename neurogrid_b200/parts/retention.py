@@ -63,8 +63,8 @@ class Retention:
         p = ctx.ws.buf("ret_in", n, self.w_in.shape[0], self.dtype)
         ops.linear(x, self.w_in, None, p)
         pa = PositionArgs.of(self.position.kernel_args())
-        if pa.inv_freq is not None and (not pa.half_pairing or pa.pos_scale != 1.0):
-            raise NotImplementedError("the retention kernel rotates pairs (i, i + dims/2) of unscaled positions")
+        if pa.inv_freq is not None and (not pa.half_pairing or pa.pos_scale != 1.0 or pa.magnitude != 1.0):
+            raise NotImplementedError("the retention kernel rotates pairs (i, i + dims/2) of unscaled positions, keeping lengths")
         rot = 0 if pa.inv_freq is None else (s.key_dim if pa.rotary_dims is None else pa.rotary_dims)
         o = ctx.ws.buf("ret_out", n, s.n_heads * s.value_dim, self.dtype)
         # float32 keeps the token-by-token kernel for every step: there a token's arithmetic is the same however

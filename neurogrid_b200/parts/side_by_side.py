@@ -19,14 +19,17 @@ class SideBySide:
     ``spec.combine`` "weighted": y = left_scale * left(x) + right_scale * right(x).  Both mixers end with a projection
     into the stream, so their inner activations (each times its scale, in float32, before its one rounding) lie side
     by side in one buffer and ONE product with the two output matrices side by side along the contraction (stacked
-    when bound) is the weighted sum; both parts must offer ``core``, ``inner_width`` and ``out_weight``."""
+    when bound) is the weighted sum; both parts must offer ``core``, ``inner_width`` and ``out_weight``.  Biases of the
+    two output projections, each times its side's scale, are one float32 vector ``out_bias``: added by this mixer, or,
+    when a block sets ``defer_bias``, left to the kernel that adds the result into the stream."""
 
     def __init__(self, spec, *, dtype, device, owns_cache=True):
         self.spec, self.dtype, self.device = spec, dtype, device
         kw = dict(dtype=dtype, device=device)
         self.left = registry.build("mixer", spec.left, **kw)
         self.right = registry.build("mixer", spec.right, **kw)
-        self.w_left = self.w_right = self.w_out = None
+        self.w_left = self.w_right = self.w_out = self.out_bias = self.b_out = None
+        self.defer_bias = False
         self.weighted = getattr(spec, "combine", "norm_mean") == "weighted"
         if self.weighted:
             for part in (self.left, self.right):
@@ -59,9 +62,13 @@ class SideBySide:
             part.bind({k[len(pre):]: v for k, v in t.items() if k.startswith(pre) and k not in own})
         if self.weighted:
             (wl, bl), (wr, br) = self.left.out_weight(), self.right.out_weight()
-            if bl is not None or br is not None:
-                raise ValueError("side by side: a weighted sum takes output projections without biases")
             self.w_out = torch.cat([wl, wr], dim=1).contiguous()
+            for part, b, scale in ((self.left, bl, self.spec.left_scale), (self.right, br, self.spec.right_scale)):
+                if b is not None:
+                    exact = getattr(part, "b_o_f32", None)           # the stored bias, before the compute dtype
+                    b = (b if exact is None else exact).to(**f32) * scale
+                    self.out_bias = b if self.out_bias is None else self.out_bias + b
+            self.b_out = self.out_bias.to(self.dtype).contiguous() if self.out_bias is not None else None
             for part in (self.left, self.right):             # the stacked matrix serves; the parts' own copies go
                 if hasattr(part, "drop_out_weight"):
                     part.drop_out_weight()
@@ -99,7 +106,8 @@ class SideBySide:
             inner = ctx.ws.buf("side_inner", x.shape[0], self.w_out.shape[1], self.dtype)
             self.left.core(x, ctx, self._views(self.left.cache_need(), views[:n_left]), inner[:, :ka], out_scale=s.left_scale)
             self.right.core(x, ctx, self._views(self.right.cache_need(), views[n_left:]), inner[:, ka:], out_scale=s.right_scale)
-            return ops.linear_to_residual(inner, self.w_out, None, ctx.ws, "mixer_out", residual=ctx.residual)
+            return ops.linear_to_residual(inner, self.w_out, None if self.defer_bias else self.b_out, ctx.ws, "mixer_out",
+                                          residual=ctx.residual)
         residual, ctx.residual = ctx.residual, None        # the parts hand their outputs over; the sum is formed here
         try:
             a = self.left.forward(x, ctx, self._views(self.left.cache_need(), views[:n_left]), out_name="side_left")

@@ -1,4 +1,4 @@
-"""Gated feed-forward: down( act(gate x) * up x ), act = silu (SwiGLU) or the tanh form of gelu."""
+"""Gated feed-forward: down( act(gate x) * up x ), act = silu (SwiGLU) or the tanh form of gelu, or both halves clamped."""
 from __future__ import annotations
 
 import torch
@@ -58,10 +58,12 @@ class SwiGLU:
     def gated(self, x, ctx, act):
         """act[N, intermediate] (may be a block of columns of a wider buffer) = act(gate x) * (up x)."""
         s = self.spec
-        activation = getattr(s, "activation", "silu")
+        kw = dict(activation=getattr(s, "activation", "silu"))
+        if kw["activation"] == "clamped_glu":
+            kw.update(limit=s.limit, alpha=s.glu_alpha)
         if ops.gemm_sm100_ok(x, self.w_gate_up):
-            ops.gemm_swiglu_sm100(x, self.w_gate_up, act, activation=activation)    # the gate rides in the epilogue
+            ops.gemm_swiglu_sm100(x, self.w_gate_up, act, **kw)    # the gate rides in the epilogue
         else:
             gu = ctx.ws.buf("ffn_gate_up", x.shape[0], 2 * s.intermediate, self.dtype)
             ops.linear(x, self.w_gate_up, None, gu)
-            ops.swiglu(gu, act, activation)
+            ops.swiglu(gu, act, **kw)

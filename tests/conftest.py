@@ -73,6 +73,14 @@ def fuzelorn_dirs(tmp_path_factory):
 
 
 @pytest.fixture(scope="session")
+def matepel_dirs(tmp_path_factory):
+    """Model folders for the tiny Matepel configurations."""
+    import matepel_models
+    return {name: matepel_models.write_model(cfg, seed, str(tmp_path_factory.mktemp(f"matepel_{name}")))
+            for name, (cfg, seed) in matepel_models.CONFIGS.items()}
+
+
+@pytest.fixture(scope="session")
 def dodilix_dirs(tmp_path_factory):
     """Model folders for the tiny Dodilix configurations; in "<name>_calm" a layer's routed experts are all alike, for
     comparisons in bfloat16 (a router's close call then changes nothing)."""

@@ -25,6 +25,12 @@ def embed(table, tokens, out, status, accumulate=False, scale=1.0):
     out.copy_(out + rows if accumulate else rows)
 
 
+def embed_norm(table, tokens, weight, out, status, eps, scale=1.0):
+    embed(table, tokens, out, status, scale=scale)
+    x = out.to(D)
+    out.copy_((x * torch.rsqrt((x * x).mean(-1, keepdim=True) + eps) * weight.to(D)).to(out.dtype))
+
+
 def gather_tokens(dst, src, idx):
     m = idx >= 0
     dst[m] = src[idx[m].long()]
@@ -47,9 +53,13 @@ def residual_add(h, delta):
     h.copy_((h.to(D) + delta.to(D)).to(torch.float32))
 
 
-def swiglu(gate_up, out, activation="silu"):
+def swiglu(gate_up, out, activation="silu", limit=0.0, alpha=0.0):
     I = out.shape[1]
     g, u = gate_up[:, :I].to(D), gate_up[:, I:].to(D)
+    if activation == "clamped_glu":
+        g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+        out.copy_((g * torch.sigmoid(alpha * g) * (u + 1)).to(out.dtype))
+        return
     if activation == "gelu_tanh":
         a = 0.5 * g * (1 + torch.tanh(math.sqrt(2 / math.pi) * (g + 0.044715 * g ** 3)))
     else:
@@ -72,12 +82,14 @@ def add_layernorm(h, delta, weight, out, eps, rows=None, post=None):
 
 
 def qkv_prep(qkv, q_out, q_weight, k_weight, inv_freq, k_pages, v_pages, table, positions, row_entry, n_q, n_k, n_v,
-             dim, vdim, eps, status, *, whole=False, q_temp_coef=0.0, q_temp_every=1, half_pairing=False, unit_norm=False):
+             dim, vdim, eps, status, *, whole=False, q_temp_coef=0.0, q_temp_every=1, half_pairing=False, unit_norm=False,
+             v_is_k=False, rot_mag=1.0):
     n = qkv.shape[0]
     x = qkv.to(D)
     q = x[:, : n_q * dim].reshape(n, n_q, dim)
     k = x[:, n_q * dim:(n_q + n_k) * dim].reshape(n, n_k, dim)
-    v = x[:, (n_q + n_k) * dim:(n_q + n_k) * dim + n_v * vdim].reshape(n, n_v, vdim)      # columns behind v are the caller's
+    v_at = (n_q if v_is_k else n_q + n_k) * dim                   # columns behind v are the caller's
+    v = x[:, v_at:v_at + n_v * vdim].reshape(n, n_v, vdim)
 
     def norm(t, w):
         if w is None and unit_norm:
@@ -94,7 +106,7 @@ def qkv_prep(qkv, q_out, q_weight, k_weight, inv_freq, k_pages, v_pages, table, 
             return t
         r = 2 * inv_freq.numel()
         ang = (positions.to(torch.float32)[:, None] * inv_freq[None, :]).to(D)          # float32 angle
-        c, s = torch.cos(ang)[:, None, :], torch.sin(ang)[:, None, :]
+        c, s = rot_mag * torch.cos(ang)[:, None, :], rot_mag * torch.sin(ang)[:, None, :]
         o = t.clone()
         if half_pairing:
             a, b = t[..., :r // 2], t[..., r // 2:r]
@@ -436,12 +448,14 @@ def gate_mul(y, gate, activation="sigmoid", scale=1.0):
 
 
 def hc_step(streams, n_streams, *, x0=None, delta=None, mix=None, out_w=None, in_w=None, norm_w=None, out=None, sum_out=None,
-            eps=0.0, act_dtype=None):
+            eps=0.0, act_dtype=None, bias=None):
     n, S = streams.shape[0], n_streams
     H = streams.shape[1] // S
     X = x0.to(D)[:, None, :].expand(n, S, H).clone() if x0 is not None else streams.to(D).reshape(n, S, H)
     if delta is not None:
         y = (delta.sum(0) if delta.dim() == 3 else delta).to(D)
+        if bias is not None:
+            y = y + bias.to(D)
         X = torch.einsum("st,nsh->nth", mix.to(D).reshape(S, S), X) + out_w.to(D)[None, :, None] * y[:, None, :]
     if x0 is not None or delta is not None:
         streams.copy_(X.reshape(n, S * H).to(streams.dtype))
@@ -482,6 +496,62 @@ def gated_linear(x, z, norm_w, state, out, cu_q, ctx_before, slots, n_entries, n
             out[r] = o.reshape(-1).to(out.dtype)
         if r1 > r0:
             state[slot] = S.to(state.dtype)
+
+
+def _norm_gate(o, group, norm_w, gate, eps, out_scale):
+    """o [nH, dv] normed over groups of ``group`` of its values in a row, weighted, gated."""
+    flat = o.reshape(-1, group)
+    flat = flat * torch.rsqrt((flat * flat).mean(-1, keepdim=True) + eps)
+    return flat.reshape(-1) * norm_w.to(D) * torch.sigmoid(gate) * out_scale
+
+
+def lightning(x, decay, norm_w, state, o_raw, out, cu_q, ctx_before, slots, row_entry, n_entries, n_heads, key_dim, value_dim,
+              eps, out_scale=1.0, scratch=None, max_q=0):
+    H, dk, dv = n_heads, key_dim, value_dim
+    act = lambda t: (t * torch.sigmoid(t)).to(x.dtype).to(D)              # rounded to the activation type
+    for e in range(n_entries):
+        r0, r1 = int(cu_q[e]), int(cu_q[e + 1])
+        slot = int(slots[e])
+        S = state[slot].to(D).clone() if int(ctx_before[e]) > 0 else torch.zeros(H, dk, dv, dtype=D, device=x.device)
+        for r in range(r0, r1):
+            row = x[r].to(D)
+            q, k = act(row[:H * dk]).reshape(H, dk), act(row[H * dk:2 * H * dk]).reshape(H, dk)
+            v = act(row[2 * H * dk:2 * H * dk + H * dv]).reshape(H, dv)
+            S = decay.to(D)[:, None, None] * S + k[:, :, None] * v[:, None, :]
+            o = torch.einsum("hkv,hk->hv", S, q)
+            out[r] = _norm_gate(o, H * dv, norm_w, row[2 * H * dk + H * dv:], eps, out_scale).to(out.dtype)
+        if r1 > r0:
+            state[slot] = S.to(state.dtype)
+
+
+def mlstm(x, gates, gate_bias, cap, norm_w, state, nm_state, o_raw, out, cu_q, ctx_before, slots, row_entry, n_entries,
+          n_heads, key_dim, value_dim, eps, out_scale=1.0, scratch=None, max_q=0):
+    H, dk, dv = n_heads, key_dim, value_dim
+    pre = cap * torch.tanh((gates.to(D) + gate_bias.to(D)) / cap)
+    log_i, log_f = pre[:, :H], torch.nn.functional.logsigmoid(pre[:, H:])
+    z = lambda *s: torch.zeros(*s, dtype=D, device=x.device)
+    for e in range(n_entries):
+        r0, r1 = int(cu_q[e]), int(cu_q[e + 1])
+        slot = int(slots[e])
+        S, n, m = z(H, dk, dv), z(H, dk), z(H)
+        if int(ctx_before[e]) > 0:
+            S, n, m = state[slot].to(D).clone(), nm_state[slot, :, 0, :dk].to(D).clone(), nm_state[slot, :, 0, dk].to(D).clone()
+        for r in range(r0, r1):
+            row = x[r].to(D)
+            q = row[:H * dk].reshape(H, dk) * dk ** -0.5
+            k = row[H * dk:2 * H * dk].reshape(H, dk)
+            v = row[2 * H * dk:2 * H * dk + H * dv].reshape(H, dv)
+            new = torch.maximum(log_f[r] + m, log_i[r])
+            keep, add = torch.exp(log_f[r] + m - new), torch.exp(log_i[r] - new)
+            S = keep[:, None, None] * S + add[:, None, None] * k[:, :, None] * v[:, None, :]
+            n, m = keep[:, None] * n + add[:, None] * k, new
+            den = torch.maximum((n * q).sum(-1).abs(), torch.exp(-m)) + 1e-6
+            o = torch.einsum("hkv,hk->hv", S, q) / den[:, None]
+            out[r] = _norm_gate(o, dv, norm_w, row[2 * H * dk + H * dv:], eps, out_scale).to(out.dtype)
+        if r1 > r0:
+            state[slot] = S.to(state.dtype)
+            nm_state[slot, :, :, :dk] = n.to(state.dtype)[:, None, :]
+            nm_state[slot, :, :, dk] = m.to(state.dtype)[:, None]
 
 
 def latent_prep(x, wq, wkv, cq_out, pages, gate_out, table, positions, row_entry, n_heads, eps, status, *, rot=0,
@@ -561,7 +631,7 @@ def head_up_gate(o, w, gate, out):
     out.copy_(y.to(out.dtype))
 
 
-_NAMES = ["scale_", "gate_mul", "hc_step", "moe_swiglu_scaled", "gated_linear", "latent_prep", "latent_rope_q", "latent_core",
+_NAMES = ["embed_norm", "lightning", "mlstm", "scale_", "gate_mul", "hc_step", "moe_swiglu_scaled", "gated_linear", "latent_prep", "latent_rope_q", "latent_core",
           "head_up_gate", "gather_tokens", "embed", "add_rmsnorm", "residual_add", "swiglu", "gemm_f32", "linear", "shortconv", "rope_cache",
           "attention_generic", "sample", "add_layernorm", "qkv_prep", "mapped_attention", "gated_delta", "pair_embed",
           "pair_norm_mean", "relu_squared_", "softcap_", "moe_router_sigmoid", "moe_clamped_glu_scaled"]
