@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the LFM2-1.2B shape, random weights, one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers N] [--impl ours|reference]
-                    [--shape 1.2b|700m|350m] [--prompt-len N] [--workload mixed350m|long700m|metanex|rofulorn|fuzelorn|dodilix]
+                    [--shape 1.2b|700m|350m] [--prompt-len N] [--workload mixed350m|long700m|metanex|rofulorn|fuzelorn|dodilix|matepel]
 
 A "step" is one decode step of the batch.  The default run has the layer sizes of the
 LFM2-1.2B configuration, a batch of 8 and requests that hold 2,048-token prompts and grow
@@ -1316,6 +1316,168 @@ def dodilix_kernel_times(eng, l2, pk):
     return out
 
 
+# ---------------------------------------------------------------------------------------------- --workload matepel
+def matepel_config(width, layers):
+    """A Matepel configuration with layers of a real model's sizes: four copies of the stream; layers alternate between
+    lightning attention (heads of 128 x 128, decays from 1/2 to nearly 1) and a parallel mixer (causal attention whose
+    values are its keys, heads of 128 with half of each head rotated and its frequencies rescaled, four query heads to a
+    key/value head, beside an mLSTM with as many heads of 128 x 128); every feed-forward dense and four widths wide."""
+    heads = width // 128
+    light = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-1 - 9 * h / max(1, heads - 1)) for h in range(heads)]}
+    left = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+            "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
+    right = {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 12.0}
+    mlp = {"kind": "dense", "ff": 4 * width, "limit": 5.0}
+    par = {"left": left, "right": right, "left_scale": 0.9, "right_scale": 1.2}
+    return {"architecture": "Matepel", "vocab": 65536, "width": width, "streams": 4, "residual_mult": 0.8, "norm": {"eps": 1e-5},
+            "layers": [{"type": "parallel", "mixer": par, "mlp": mlp} if i % 2 else {"type": "lightning", "mixer": light, "mlp": mlp}
+                       for i in range(layers)]}
+
+
+def run_matepel(args):
+    """Prefill and decode throughput of the Matepel design at layer sizes of a real model, beside Dodilix (the closest
+    existing model: copies of the stream, an attention with float32 weights beside a linear attention with a float32
+    state) at equal width and depth, and both designs' own kernels one by one.  One JSON line.  Random weights,
+    synthetic token ids; CUDA events; the L2 is flushed between timed steps."""
+    import torch
+    pk = peaks()
+    l2 = torch.zeros(256 << 20, dtype=torch.uint8, device="cuda:0")
+    clocks = ClockSampler(0)
+    clocks.start()
+    results = []
+    for width, layers in ((1024, 16), (2048, 16)):
+        row = {"width": width, "layers": layers}
+        for arm, cfg in {"matepel": matepel_config(width, layers), "dodilix": dodilix_config(width, layers)}.items():
+            eng = design_arm(arm, cfg, row, args, l2)
+            if not args.no_kernels:
+                row[arm + "_kernels"] = (matepel_kernel_times if arm == "matepel" else dodilix_kernel_times)(eng, l2, pk)
+            del eng
+            torch.cuda.empty_cache()
+        results.append(row)
+    time.sleep(0.06)
+    clocks.stop()
+    print(json.dumps({"workload": "matepel", "what": "Matepel beside Dodilix at equal width and depth: prefill of 2,048 "
+                      "tokens, decode at batch 8 and 1 after 2,048 tokens; each design's own kernels alone",
+                      "results": results, "dtype": "bf16", "data": "synthetic token ids, random-init weights", "peaks": pk,
+                      "clocks": clocks.summary(), "impl": "ours"}))
+
+
+def matepel_kernel_times(eng, l2, pk):
+    """The design's own kernels alone, through the parts' own launch plans (CUDA events around the launches, L2 flushed
+    before, median of 7), for a 2,048-token portion and for 8 single tokens after 2,048: microseconds, the bytes each
+    must move with the fraction of the measured copy bandwidth, and for the recurrences and the attention core the
+    multiply-adds they must do as TFLOP/s."""
+    import torch
+    from neurogrid_b200.csrc import ops
+    from neurogrid_b200.parts import PagedView, StepContext
+    from neurogrid_b200.parts.base import Workspace
+    model, dev = eng.model, eng.device
+    D, S = model.spec.hidden, model.spec.streams
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    g = torch.Generator(device=dev).manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev).to(torch.bfloat16)
+
+    def timed(fn):
+        ts = []
+        for _ in range(9):
+            flush_l2(l2)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b) * 1e3)
+        return median(ts[2:])
+
+    out = {"unit": "us"}
+    bw = pk["hbm_gbs"] * 1e9
+
+    def mem(name, us, nbytes, flops=0):
+        out[name] = {"us": round(us, 2), "bytes": int(nbytes), "of_copy_bandwidth": round(nbytes / (us * 1e-6) / bw, 3)}
+        if flops:
+            out[name]["flops"] = int(flops)
+            out[name]["tflops"] = round(flops / (us * 1e-6) / 1e12, 2)
+
+    par = next(b for b in model.blocks if type(b.mixer).__name__ == "SideBySide")
+    light = next(b.mixer for b in model.blocks if type(b.mixer).__name__ == "LightningAttention")
+    side, f = par.mixer, par.ffn
+    left, right = side.left, side.right
+    ls, rs, gs = left.spec, right.spec, light.spec
+    need = left.cache_need()
+    ps, n_pages = 16, 8 * 4096 // 16
+    kp, vp = (rnd(n_pages, need.n_kv_heads, ps, need.head_dim) for _ in range(2))
+    for rows, entries in ((PREFILL_TOKENS, 1), (8, 8)):
+        tag = "prefill2048" if entries == 1 else "decode8"
+        q_len = rows // entries
+        before = 0 if entries == 1 else 2048
+        table = torch.arange(entries * 256, dtype=torch.int32, device=dev).view(entries, 256)
+        ctx = StepContext(n_rows=rows, n_entries=entries, max_q=q_len, tokens=i32([(7 * t) % 999 for t in range(rows)]),
+                          positions=i32([before + t for e in range(entries) for t in range(q_len)]),
+                          row_entry=i32([e for e in range(entries) for _ in range(q_len)]),
+                          cu_q=i32([q_len * e for e in range(entries + 1)]), ctx_before=i32([before] * entries),
+                          slots=i32(list(range(entries))), status=torch.zeros(1, dtype=torch.int32, device=dev),
+                          ws=Workspace(4096, dev), dtype=torch.bfloat16, q_lens=[q_len] * entries,
+                          ctx_lens=[before] * entries, slot_ids=list(range(entries)))
+        # the embedding with its norm
+        h = torch.empty(rows, D, device=dev)
+        us = timed(lambda: ops.embed_norm(model.embed_table, ctx.tokens, model.embed_norm.weight, h, ctx.status, 1e-5))
+        mem(f"{tag}_embed_norm", us, rows * D * (2 + 4))
+        # between two sublayers: the copies' update (with the mixer's bias), the read-out and its norm
+        X, y = torch.randn(rows, S * D, generator=g, device=dev), rnd(rows, D)
+        w_in, w_out, mix = par.hc["hc1"]
+        normed = torch.empty(rows, D, dtype=torch.bfloat16, device=dev)
+        us = timed(lambda: ops.hc_step(X, S, delta=y, mix=mix, out_w=w_out, in_w=w_in, norm_w=par.mixer_norm.weight, out=normed,
+                                       eps=1e-5, bias=side.out_bias))
+        mem(f"{tag}_stream_copies", us, rows * D * (2 * 4 * S + 2 + 2))
+        # left: rotation and page write; the attention core
+        d, H, G = ls.key_dim, ls.n_heads, need.n_kv_heads
+        qk = rnd(rows, left.w_qkv.shape[0])
+        qb = torch.empty(rows, H * d, dtype=torch.bfloat16, device=dev)
+        pa = left.position.kernel_args()
+        view = PagedView(kp, vp, table)
+        o = torch.empty(rows, H * d, dtype=torch.bfloat16, device=dev)
+        prep = lambda: ops.qkv_prep(qk, qb, None, None, pa.inv_freq, kp, vp, table, ctx.positions, ctx.row_entry, H, G, G, d, d,
+                                    ls.eps, ctx.status, half_pairing=True, v_is_k=True, rot_mag=pa.magnitude)
+        core = lambda: left.attend(qb, view, ctx, o, None)
+        prep()
+        core()
+        torch.cuda.synchronize()
+        mem(f"{tag}_attention_prep", timed(prep), (2 * H + 3 * G) * d * rows * 2)
+        pairs = sum(t + 1 for t in range(rows)) if entries == 1 else rows * (before + 1)
+        us = timed(core)
+        mem(f"{tag}_attention_core", us, entries * (before + q_len) * need.elements_per_token() * 2 + 2 * rows * H * d * 2,
+            4 * pairs * H * d)
+        out[f"{tag}_attention_core"]["of_tensor_peak"] = round(4 * pairs * H * d / (us * 1e-6) / 1e12 / pk["bf16_tflops"], 4)
+        # the recurrences with their gates, norms and output gates (one call of a part's launcher each)
+        for part, spec, name in ((right, rs, "mlstm"), (light, gs, "lightning")):
+            nH, dk, dv = spec.n_heads, spec.key_dim, spec.value_dim
+            p = rnd(rows, part.w_in.shape[0])
+            state = torch.zeros(8, nH, dk, dv, device=dev)
+            raw, og = torch.empty(rows, nH * dv, device=dev), torch.empty(rows, nH * dv, dtype=torch.bfloat16, device=dev)
+            scratch = part._chunk_scratch(ctx, rows)         # as the part chooses: long portions chunk by chunk
+            tail = (raw, og, ctx.cu_q, ctx.ctx_before, ctx.slots, ctx.row_entry, entries, nH, dk, dv, spec.eps, 1.0)
+            kw = dict(scratch=scratch, max_q=q_len)
+            if name == "mlstm":
+                gates = torch.randn(rows, 2 * nH, generator=g, device=dev)
+                nm = torch.zeros(8, nH, ops.decayed_linear_slices(dv), dk + 1, device=dev)
+                run = lambda: ops.mlstm(p, gates, part.b_gates, spec.gate_cap, part.norm, state, nm, *tail, **kw)
+                xs = rnd(rows, D)
+                mem(f"{tag}_mlstm_gate_product", timed(lambda: ops.linear(xs, part.w_gates, None, gates)),
+                    rows * D * 2 + part.w_gates.numel() * 2 + gates.numel() * 4)
+            else:
+                run = lambda: ops.lightning(p, part.decay, part.norm, state, *tail, **kw)
+            run()
+            torch.cuda.synchronize()
+            mem(f"{tag}_{name}", timed(run), (p.numel() + og.numel()) * 2 + 2 * entries * state[0].numel() * 4,
+                4 * rows * nH * dk * dv)
+        # the clamped gate behind the library's product of a long step (in a short one it rides in the product)
+        if entries == 1:
+            I = f.spec.intermediate
+            gu, act = rnd(rows, 2 * I), torch.empty(rows, I, dtype=torch.bfloat16, device=dev)
+            mem(f"{tag}_clamped_gate", timed(lambda: ops.swiglu(gu, act, "clamped_glu", f.spec.limit, f.spec.glu_alpha)), 3 * rows * I * 2)
+    return out
+
+
 def run_reference(args):
     """The reference's own library through its stock entry points; same metric, same line."""
     shape_name = SHAPE_NAMES[args.shape]
@@ -1378,7 +1540,7 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=0,
                     help="tokens each request holds before decoding (default 2,048; the context is twice this)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="", choices=["", "mixed350m", "long700m", "metanex", "rofulorn", "fuzelorn", "dodilix"],
+    ap.add_argument("--workload", default="", choices=["", "mixed350m", "long700m", "metanex", "rofulorn", "fuzelorn", "dodilix", "matepel"],
                     help="run another workload of the benchmark set through Engine.generate instead; metanex / rofulorn: "
                          "that design beside LFM2 at equal width and depth, prefill and decode, and its kernels alone")
     ap.add_argument("--repeat", type=int, default=2, help="--workload: runs (the first also warms up and captures graphs)")
@@ -1397,6 +1559,9 @@ def main():
         args.warmup = 3
     if args.workload == "metanex":
         run_metanex(args)
+        return 0
+    if args.workload == "matepel":
+        run_matepel(args)
         return 0
     if args.workload == "dodilix":
         run_dodilix(args)

@@ -51,11 +51,14 @@ struct DlGeom {
 };
 
 __device__ __forceinline__ float dl_silu(float z) { return z / (1.f + expf(-z)); }
-// silu rounded to the activation type: what a projection with its activation would store
+// silu as the activation type holds it: what a projection with its activation would store (bfloat16: through the fast
+// exponential and division, whose errors are far below that rounding)
+__device__ __forceinline__ float dl_silu_fast(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 template <typename T>
 __device__ __forceinline__ float dl_silu_as(float z) {
+    if (sizeof(T) == 4) return dl_silu(z);
     T r;
-    ng_st(&r, dl_silu(z));
+    ng_st(&r, dl_silu_fast(z));
     return ng_ld(&r);
 }
 __device__ __forceinline__ float dl_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
@@ -111,7 +114,7 @@ dl_step_kernel(const T* __restrict__ x, const float* __restrict__ gates, const f
     const float* gt = ng_after_wait(gates);
     const size_t ld = 2 * (size_t)nH * (dk + dv);
     const size_t off_q = (size_t)head * dk, off_k = (size_t)nH * dk + off_q, off_v = 2 * (size_t)nH * dk + (size_t)head * dv;
-    const float lam = MODE == DL_LIGHTNING ? decay[head] : 0.f;
+    const float lam = MODE == DL_LIGHTNING ? decay[head * (DC + 1) + 1] : 0.f;
     const float qscale = MODE == DL_MLSTM ? rsqrtf((float)dk) : 1.f;
     for (int t0 = 0; t0 < qlen; t0 += DL_TOKENS) {
         const int nt = min(DL_TOKENS, qlen - t0);
@@ -231,6 +234,66 @@ dl_finish_kernel(const float* __restrict__ o, const T* __restrict__ gate, const 
     }
 }
 
+// The same in one pass over memory: four columns a thread and step, at most NV steps, all loads issued before the norm's
+// sum.  A warp per (row, group), or (WHOLE) a block per row whose columns are one group.
+__device__ __forceinline__ float4 dl_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 dl_ld4(const bf16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void dl_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void dl_st4(bf16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <typename T, bool WHOLE, int NV>
+__global__ void __launch_bounds__(512)
+dl_finish_vec_kernel(const float* __restrict__ o, const T* __restrict__ gate, const float* __restrict__ w, T* __restrict__ out,
+                     const int* __restrict__ row_entry, int n_rows, int width, int group, int ldg, int ldo, float eps, float scale) {
+    __shared__ float red[32];
+    ng_pdl_trigger();
+    const int groups = width / group;
+    const size_t unit = WHOLE ? blockIdx.x : (size_t)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int me = WHOLE ? threadIdx.x : threadIdx.x & 31, step = 4 * (WHOLE ? blockDim.x : 32);
+    const bool mine = unit < (size_t)n_rows * groups;
+    const size_t row = mine ? unit / groups : 0;
+    const int c0 = (int)(unit % groups) * group;
+    float4 wv[NV];
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = 4 * me + k * step;
+        wv[k] = mine && c < group ? dl_ld4(w + c0 + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    ng_pdl_wait();
+    if (!mine) return;                                 // (WHOLE: never; else a whole warp)
+    const float* in = ng_after_wait(o) + row * (size_t)width + c0;
+    const T* gr = ng_after_wait(gate) + row * (size_t)ldg + c0;
+    const bool real = row_entry[row] >= 0;             // padding row: zeros
+    float4 v[NV], g[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = 4 * me + k * step;
+        v[k] = g[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (real && c < group) { v[k] = dl_ld4(in + c); g[k] = dl_ld4(gr + c); }
+    }
+#pragma unroll
+    for (int k = 0; k < NV; ++k) ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    ss = WHOLE ? ng_block_sum(ss, red) : ng_warp_sum(ss);
+    const float r = rsqrtf(ss / (float)group + eps);
+    T* orow = out + row * (size_t)ldo + c0;
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+        const int c = 4 * me + k * step;
+        if (c < group)
+            dl_st4(orow + c, make_float4(v[k].x * r * wv[k].x * (scale / (1.f + expf(-g[k].x))),
+                                         v[k].y * r * wv[k].y * (scale / (1.f + expf(-g[k].y))),
+                                         v[k].z * r * wv[k].z * (scale / (1.f + expf(-g[k].z))),
+                                         v[k].w * r * wv[k].w * (scale / (1.f + expf(-g[k].w)))));
+    }
+}
+
 // -------------------------------------------------------------------------------------------- chunk by chunk
 __device__ __forceinline__ void dl_ldsm_x4(uint32_t (&r)[4], const void* p) {
     const uint32_t a = (uint32_t)__cvta_generic_to_shared(p);
@@ -259,6 +322,25 @@ __device__ __forceinline__ void dl_split3(float x, float y, uint32_t& hi, uint32
     lo = dl_pack(xr - __uint_as_float(mid << 16), yr - __uint_as_float(mid & 0xffff0000u));
 }
 
+// acc[16 x N] += (hi + mid + lo)[16 x 16] v[16 x N], v in shared memory (`v`: this lane's row and column of the first
+// group of 16 columns); smallest terms first, the column groups taking turns so that an accumulator's products are apart
+template <int N>
+__device__ __forceinline__ void dl_add_split(float (&acc)[N / 8][4], const uint32_t (&hi)[4], const uint32_t (&mid)[4],
+                                             const uint32_t (&lo)[4], const bf16* v) {
+    uint32_t b[N / 16][4];
+#pragma unroll
+    for (int x = 0; x < N / 16; ++x) dl_ldsm_x4_t(b[x], v + x * 16);
+#pragma unroll
+    for (int term = 0; term < 3; ++term) {
+        const uint32_t (&a)[4] = term == 0 ? lo : term == 1 ? mid : hi;
+#pragma unroll
+        for (int x = 0; x < N / 16; ++x) {
+            dl_mma(acc[2 * x], a, b[x][0], b[x][1]);
+            dl_mma(acc[2 * x + 1], a, b[x][2], b[x][3]);
+        }
+    }
+}
+
 // columns [c0, c0 + cols) of n rows (64 at most; the rest zero) into shared memory, 16 bytes at a time, silu applied
 // for lightning; dst row pitch `pitch` elements
 template <int MODE>
@@ -273,7 +355,7 @@ __device__ __forceinline__ void dl_load_tile(bf16* dst, int pitch, const bf16* _
                 uint32_t* u = reinterpret_cast<uint32_t*>(&v);
 #pragma unroll
                 for (int k = 0; k < 4; ++k)
-                    u[k] = dl_pack(dl_silu(__uint_as_float(u[k] << 16)), dl_silu(__uint_as_float(u[k] & 0xffff0000u)));
+                    u[k] = dl_pack(dl_silu_fast(__uint_as_float(u[k] << 16)), dl_silu_fast(__uint_as_float(u[k] & 0xffff0000u)));
             }
         }
         *reinterpret_cast<uint4*>(dst + t * pitch + c) = v;
@@ -359,17 +441,6 @@ dl_gates_kernel(const float* __restrict__ gates, const float* __restrict__ gate_
     for (int k = threadIdx.x; k < slices; k += blockDim.x) nm[(size_t)k * (dk + 1)] = m0;
 }
 
-// powers lambda^0 .. lambda^DC into shared memory, by repeated multiplication
-__device__ __forceinline__ void dl_powers(float* pw, float lam) {
-    if (threadIdx.x == 0) {
-        float p = 1.f;
-        for (int n = 0; n <= DC; ++n) {
-            pw[n] = p;
-            p *= lam;
-        }
-    }
-}
-
 // U of a chunk for one head and slice of DVS value columns (and, slice 0 of the mLSTM, the same sum without v)
 template <int MODE, int DVS>
 __global__ void __launch_bounds__(DC_THREADS)
@@ -380,7 +451,7 @@ dl_local_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, cons
     constexpr int VP = DVS + 8;
     bf16* Ks = reinterpret_cast<bf16*>(smem_raw);      // [DC][KP]
     bf16* Vs = Ks + DC * KP;                           // [DC][VP]
-    __shared__ float ws[DC], pw[DC + 1];
+    __shared__ float ws[DC];
     ng_pdl_trigger();
     ng_pdl_wait();
     const int c = blockIdx.x, e = blockIdx.y, slices = dv / DVS;
@@ -394,9 +465,7 @@ dl_local_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, cons
     dl_load_tile<MODE>(Ks, KP, xr + (size_t)nH * dk + (size_t)head * dk, ld, dk, n);
     dl_load_tile<MODE>(Vs, VP, xr + 2 * (size_t)nH * dk + (size_t)head * dv + sl * DVS, ld, DVS, n);
     if (MODE == DL_LIGHTNING) {
-        dl_powers(pw, decay[head]);
-        __syncthreads();
-        if (tid < DC) ws[tid] = tid < n ? pw[n - 1 - tid] : 0.f;
+        if (tid < DC) ws[tid] = tid < n ? decay[head * (DC + 1) + n - 1 - tid] : 0.f;
     } else if (tid < DC) {
         const float a_last = tok[(size_t)(row0 + n - 1) * nH + head].x;
         ws[tid] = tid < n ? expf(a_last - tok[(size_t)(row0 + tid) * nH + head].y) : 0.f;
@@ -419,17 +488,7 @@ dl_local_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, cons
                 const int t = kk * 16 + 2 * tq + (u >> 1) * 8;
                 dl_split3(__uint_as_float(a[u] << 16) * ws[t], __uint_as_float(a[u] & 0xffff0000u) * ws[t + 1], ah[u], am[u], al[u]);
             }
-#pragma unroll
-            for (int np = 0; np < DVS / 16; ++np) {
-                uint32_t b[4];
-                dl_ldsm_x4_t(b, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + np * 16 + (lane >> 4) * 8);
-                dl_mma(acc[2 * np], al, b[0], b[1]);
-                dl_mma(acc[2 * np + 1], al, b[2], b[3]);
-                dl_mma(acc[2 * np], am, b[0], b[1]);
-                dl_mma(acc[2 * np + 1], am, b[2], b[3]);
-                dl_mma(acc[2 * np], ah, b[0], b[1]);
-                dl_mma(acc[2 * np + 1], ah, b[2], b[3]);
-            }
+            dl_add_split<DVS>(acc, ah, am, al, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + (lane >> 4) * 8);
         }
 #pragma unroll
         for (int j = 0; j < DVS / 8; ++j) {
@@ -478,12 +537,8 @@ dl_scan_kernel(float* __restrict__ u_scratch, float* __restrict__ un_scratch, fl
     const int nc = (qlen + DC - 1) / DC;
     float full = 1.f, last = 1.f;
     if (MODE == DL_LIGHTNING) {
-        const float lam = decay[head];
-        const int rest = qlen - (nc - 1) * DC;
-        for (int k = 0; k < DC; ++k) {
-            full *= lam;
-            if (k == rest - 1) last = full;
-        }
+        full = decay[head * (DC + 1) + DC];
+        last = decay[head * (DC + 1) + qlen - (nc - 1) * DC];
     }
     for (int c0 = 0; c0 < nc; c0 += AHEAD) {
         float4 u[AHEAD];
@@ -570,7 +625,8 @@ dl_out_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, const 
     }
     const float scale = MODE == DL_MLSTM ? rsqrtf((float)dk) : 1.f;
     if (MODE == DL_LIGHTNING) {
-        dl_powers(pw, decay[head]);
+        if (tid <= DC) pw[tid] = decay[head * (DC + 1) + tid];
+        if (tid < DC) ein_s[tid] = decay[head * (DC + 1) + tid + 1];
     } else {
         for (int i = tid; i < dk; i += DC_THREADS) ns[i] = un_scratch[slot * dk + i];
         if (tid < DC) {
@@ -591,10 +647,7 @@ dl_out_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, const 
         a += __shfl_xor_sync(0xffffffffu, a, 1);
         if (h == 0) nq_s[t] = a * ein_s[t];
         __syncthreads();
-    } else if (tid < DC) {
-        ein_s[tid] = pw[tid + 1];
     }
-    if (MODE == DL_LIGHTNING) __syncthreads();
     const int w0 = warp * 16;
     if (w0 >= n) return;
     const int gq = lane >> 2, tq = lane & 3;
@@ -652,17 +705,7 @@ dl_out_kernel(const bf16* __restrict__ x, const float4* __restrict__ tok, const 
         dl_split3(s[2 * kk][2], s[2 * kk][3], ah[1], am[1], al[1]);
         dl_split3(s[2 * kk + 1][0], s[2 * kk + 1][1], ah[2], am[2], al[2]);
         dl_split3(s[2 * kk + 1][2], s[2 * kk + 1][3], ah[3], am[3], al[3]);
-#pragma unroll
-        for (int np = 0; np < DVS / 16; ++np) {
-            uint32_t b[4];
-            dl_ldsm_x4_t(b, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + np * 16 + (lane >> 4) * 8);
-            dl_mma(o[2 * np], al, b[0], b[1]);
-            dl_mma(o[2 * np + 1], al, b[2], b[3]);
-            dl_mma(o[2 * np], am, b[0], b[1]);
-            dl_mma(o[2 * np + 1], am, b[2], b[3]);
-            dl_mma(o[2 * np], ah, b[0], b[1]);
-            dl_mma(o[2 * np + 1], ah, b[2], b[3]);
-        }
+        dl_add_split<DVS>(o, ah, am, al, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + (lane >> 4) * 8);
     }
     float ra = 1.f, rb = 1.f;
     if (MODE == DL_MLSTM) {
@@ -705,7 +748,8 @@ static int dl_step(const void* x, const float* gates, const float* gate_bias, co
     return ng_launch_status();
 }
 
-// Token by token.  x [n_rows, 2 nH (dk + dv)]; lightning (gates null): decay [nH]; mLSTM: gates [n_rows, 2 nH] float32
+// Token by token.  x [n_rows, 2 nH (dk + dv)]; lightning (gates null): decay [nH][DC + 1], the powers of every head's
+// decay; mLSTM: gates [n_rows, 2 nH] float32
 // preactivations i | f, gate_bias [2 nH], nm_state [slots, nH, ng_dl_slices(dv), dk + 1].  o_raw float32 [n_rows, nH dv].
 NG_EXPORT int ng_dl_step(const void* x, const float* gates, const float* gate_bias, const float* decay, float cap,
                          float* state, float* nm_state, float* o_raw, const int* cu_q, const int* ctx_before,
@@ -783,6 +827,27 @@ NG_EXPORT int ng_dl_finish(const float* o_raw, const void* gate, const float* w,
                            int width, int group, int ldg, int ldo, float eps, float scale, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (width <= 0 || group <= 0 || width % group || ldg < width || ldo < width) return NG_BAD_SIZE;
+    const size_t pair = act_bf16 ? 8 : 16;             // bytes of four activations
+    const bool vec = group % 4 == 0 && ldg % 4 == 0 && ldo % 4 == 0 && ((uintptr_t)o_raw & 15) == 0 && ((uintptr_t)w & 15) == 0 &&
+                     (uintptr_t)gate % pair == 0 && (uintptr_t)out % pair == 0;
+#define DL_FINISH_VEC(TT, WH, NV, GRID, THREADS)                                                                          \
+    NG_LAUNCH((dl_finish_vec_kernel<TT, WH, NV>), (GRID), (THREADS), 0, stream, o_raw, (const TT*)gate, w, (TT*)out, row_entry, n_rows, \
+              width, group, ldg, ldo, eps, scale)
+    if (vec && group == width && width <= 8192) {      // a block per row
+        const int threads = width >= 2048 ? 512 : (width / 4 + 31) / 32 * 32;
+        const int nv = (width + 4 * threads - 1) / (4 * threads);
+        if (act_bf16) { if (nv <= 1) DL_FINISH_VEC(bf16, true, 1, n_rows, threads); else if (nv <= 2) DL_FINISH_VEC(bf16, true, 2, n_rows, threads); else DL_FINISH_VEC(bf16, true, 4, n_rows, threads); }
+        else { if (nv <= 1) DL_FINISH_VEC(float, true, 1, n_rows, threads); else if (nv <= 2) DL_FINISH_VEC(float, true, 2, n_rows, threads); else DL_FINISH_VEC(float, true, 4, n_rows, threads); }
+        return ng_launch_status();
+    }
+    if (vec && group < width && group <= 512) {        // a warp per (row, head)
+        const size_t units = (size_t)n_rows * (width / group);
+        const unsigned blocks = (unsigned)((units + 3) / 4);
+        const int nv = (group + 127) / 128;
+        if (act_bf16) { if (nv <= 1) DL_FINISH_VEC(bf16, false, 1, blocks, 128); else if (nv <= 2) DL_FINISH_VEC(bf16, false, 2, blocks, 128); else DL_FINISH_VEC(bf16, false, 4, blocks, 128); }
+        else { if (nv <= 1) DL_FINISH_VEC(float, false, 1, blocks, 128); else if (nv <= 2) DL_FINISH_VEC(float, false, 2, blocks, 128); else DL_FINISH_VEC(float, false, 4, blocks, 128); }
+        return ng_launch_status();
+    }
     if (act_bf16)
         NG_LAUNCH((dl_finish_kernel<bf16>), n_rows, 256, 0, stream, o_raw, (const bf16*)gate, w, (bf16*)out, row_entry, width, group, ldg, ldo, eps, scale);
     else

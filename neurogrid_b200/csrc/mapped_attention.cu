@@ -9,7 +9,7 @@
 //   M == 1: o = a_0                          M == 2: o = a_0 - lambda * a_1
 //   slopes (per head, optional): slope_h * (pos - j) is taken off s(j) after the cap
 //   sinks (per head, optional): the softmax's denominator also holds exp(sink_h), a term without key or value
-//   head_norm: o <- o * rsqrt(mean(o^2) + eps) * post_scale  over the head's dv values
+//   head_norm: o <- o * rsqrt(mean(o^2) + eps)  over the head's dv values;   then o <- o * post_scale
 //
 // Two kernels.  ``qkv_prep``: per-head RMS norm of q and k (one weight vector shared by heads and maps; or, `whole`,
 // one norm over all of a row's q and one over all of its k, with weights of that length), q times a temperature
@@ -253,8 +253,8 @@ __device__ __forceinline__ void ma_finish(const MaParams& p, T* o, const float* 
         keep[n] = v;
         ss += v * v;
     }
-    float r = 1.f;
-    if (p.head_norm) r = rsqrtf(ng_block_sum(ss, red) / (float)p.dv + p.eps) * p.post_scale;
+    float r = p.post_scale;
+    if (p.head_norm) r *= rsqrtf(ng_block_sum(ss, red) / (float)p.dv + p.eps);
     n = 0;
     for (int c = threadIdx.x; c < p.dv; c += MA_THREADS, ++n) ng_st(o + c, keep[n] * r);
 }
@@ -431,12 +431,13 @@ mapped_attention_kernel(const MaParams p) {
 template <typename T, int M>
 __global__ void __launch_bounds__(MA_THREADS)
 mapped_attention_merge_kernel(const MaParams p) {
-    extern __shared__ float sm[];                       // [M][dv]
+    extern __shared__ float sm[];                       // [M][dv], then the runs' factors [n_splits]
     __shared__ float red[32];
     ng_pdl_trigger();
-    ng_pdl_wait();
     const int row = blockIdx.x, head = blockIdx.y;
-    const int dv = p.dv;
+    const int dv = p.dv, lane = threadIdx.x & 31;
+    float* f_s = sm + (size_t)M * dv;
+    ng_pdl_wait();
     T* o = reinterpret_cast<T*>(p.out) + (size_t)row * p.out_ld + (size_t)head * dv;
     if (p.row_entry[row] < 0) {
         for (int c = threadIdx.x; c < dv; c += MA_THREADS) ng_st(o + c, 0.f);
@@ -446,22 +447,24 @@ mapped_attention_merge_kernel(const MaParams p) {
     float lf[M];
 #pragma unroll
     for (int m = 0; m < M; ++m) {
+        // a lane per run (32 runs at a time) for the maximum, the factors and the sum; every warp forms them itself
         float mt = -INFINITY;
-        for (int s = 0; s < p.n_splits; ++s) mt = fmaxf(mt, part[((size_t)s * M + m) * (dv + 2)]);
+        for (int s = lane; s < p.n_splits; s += 32) mt = fmaxf(mt, part[((size_t)s * M + m) * (dv + 2)]);
+        mt = ng_warp_max(mt);
         float lt = 0.f;
-        for (int s = 0; s < p.n_splits; ++s) {
+        __syncthreads();                                 // the other map's factors have been read
+        for (int s = lane; s < p.n_splits; s += 32) {
             const float* ps = part + ((size_t)s * M + m) * (dv + 2);
             const float f = ps[0] == -INFINITY ? 0.f : expf(ps[0] - mt);
+            if (threadIdx.x < 32) f_s[s] = f;
             lt += ps[1] * f;
         }
-        lf[m] = lt + (p.sinks ? expf(p.sinks[head] - mt) : 0.f);
+        lf[m] = ng_warp_sum(lt) + (p.sinks ? expf(p.sinks[head] - mt) : 0.f);
+        __syncthreads();
         for (int c = threadIdx.x; c < dv; c += MA_THREADS) {
             float a = 0.f;
-            for (int s = 0; s < p.n_splits; ++s) {
-                const float* ps = part + ((size_t)s * M + m) * (dv + 2);
-                const float f = ps[0] == -INFINITY ? 0.f : expf(ps[0] - mt);
-                a += ps[2 + c] * f;
-            }
+#pragma unroll 8
+            for (int s = 0; s < p.n_splits; ++s) a = fmaf(part[((size_t)s * M + m) * (dv + 2) + 2 + c], f_s[s], a);
             sm[(size_t)m * dv + c] = a;
         }
     }
@@ -478,8 +481,9 @@ static int ma_launch(const MaParams& p, int n_rows, cudaStream_t stream) {
     else if (p.dv <= 128) NG_LAUNCH((mapped_attention_kernel<T, M, 2>), grid, MA_THREADS, smem, stream, p);
     else NG_LAUNCH((mapped_attention_kernel<T, M, 4>), grid, MA_THREADS, smem, stream, p);
     if (p.n_splits > 1) {
+        if (((size_t)M * p.dv + p.n_splits) * sizeof(float) > 48 * 1024) return NG_BAD_SIZE;
         dim3 g2(n_rows, p.nH);
-        NG_LAUNCH((mapped_attention_merge_kernel<T, M>), g2, MA_THREADS, (size_t)M * p.dv * sizeof(float), stream, p);
+        NG_LAUNCH((mapped_attention_merge_kernel<T, M>), g2, MA_THREADS, ((size_t)M * p.dv + p.n_splits) * sizeof(float), stream, p);
     }
     return ng_launch_status();
 }
@@ -515,7 +519,8 @@ NG_EXPORT int ng_mapped_attention_merge(float* partial, const int* row_entry, vo
     MaParams p{nullptr, nullptr, nullptr, nullptr, 0, nullptr, row_entry, out, out_ld, partial, nH, 1, 0, dv, 1, 0, 0, 0, n_splits, 0,
                0.f, 0.f, lambda, post_scale, eps, head_norm, nullptr, sinks};
     dim3 grid(n_rows, nH);
-    const size_t smem = (size_t)n_maps * dv * sizeof(float);
+    const size_t smem = ((size_t)n_maps * dv + n_splits) * sizeof(float);
+    if (smem > 48 * 1024) return NG_BAD_SIZE;
     if (act_bf16) {
         if (n_maps == 2) NG_LAUNCH((mapped_attention_merge_kernel<__nv_bfloat16, 2>), grid, MA_THREADS, smem, stream, p);
         else NG_LAUNCH((mapped_attention_merge_kernel<__nv_bfloat16, 1>), grid, MA_THREADS, smem, stream, p);

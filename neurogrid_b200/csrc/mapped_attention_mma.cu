@@ -24,6 +24,7 @@ static_assert(NG_MA_DV % 16 == 0 && NG_MA_DV >= 16 && NG_MA_DV <= 128, "value si
 typedef __nv_bfloat16 bf16;
 constexpr int D = NG_MA_D, DV = NG_MA_DV;
 constexpr int KT = 64, WARPS = 4, THREADS = 128;
+constexpr int TURNS = 4;                                 // groups of 16 value columns whose products take turns
 constexpr int QP = D + 8, KP = D + 8, VP = DV + 8;      // row pitches in elements: 16 bytes of padding against bank conflicts
 
 struct MmaParams {
@@ -82,12 +83,16 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t&
 }
 
 // GROUP: for entries that bring one token.  The rows of the tile are then the query heads of one KV group (up to 16; they
-// share keys and values and here also the position), a block takes (run of keys, entry, KV group), and instead of the
-// finished heads it leaves each run's state (maximum, sum, weighted values) for the kernel that merges runs.
+// share keys and values and here also the position), a block takes (run of keys, entry, KV group), the warps of a map
+// take different keys of every tile (each keeps a softmax state of its own; merged in warp order at the end), and
+// instead of the finished heads the block leaves each run's state (maximum, sum, weighted values) for the kernel that
+// merges runs.
 template <int M, bool GROUP>
 __global__ void __launch_bounds__(THREADS, 3)
 mapped_attention_mma_kernel(const MmaParams p) {
     constexpr int ROWS = (WARPS / M) * 16;               // rows of a block
+    constexpr int PARTS = GROUP ? WARPS / M : 1;         // warps that share a tile's keys
+    constexpr int KW = KT / PARTS;                       // keys of a tile that a warp works on
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);                        // [M][ROWS][QP]
     bf16* Ks = Qs + M * ROWS * QP;                                       // [2][M][KT][KP]
@@ -95,7 +100,8 @@ mapped_attention_mma_kernel(const MmaParams p) {
     float* Os = reinterpret_cast<float*>(Ks);                            // epilogue: [M][ROWS][DV], over the tiles
     __shared__ int kpos_s[3][KT];                                        // per tile in flight or in use (three: see the loop)
     __shared__ long long koff_s[3][KT];
-    __shared__ int tile_bad_s[3][2];                                     // a key of the tile has no page                                  // element offset of the key's page slot, -1: none
+    __shared__ int tile_bad_s[3][2];                                     // a key of the tile has no page
+    __shared__ float part_m[WARPS][16], part_l[WARPS][16];               // GROUP: the warps' states per row
     ng_pdl_trigger();
     const int entry = blockIdx.y;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -109,7 +115,8 @@ mapped_attention_mma_kernel(const MmaParams p) {
     const int g = GROUP ? blockIdx.z : blockIdx.z / group_heads;
     const int head = GROUP ? g * group_heads : blockIdx.z;               // GROUP: the first head of the tile's rows
     const int map = M == 2 ? (warp & 1) : 0;
-    const int wt = M == 2 ? (warp >> 1) : warp;          // the warp's tile of 16 rows
+    const int wt = GROUP ? 0 : M == 2 ? (warp >> 1) : warp;              // the warp's tile of 16 rows
+    const int k_off = GROUP ? (M == 2 ? (warp >> 1) : warp) * KW : 0;    // ... and its first key of every tile
     const bf16* qg = ng_after_wait(p.q);
     // ---- Q: rows r0.., both maps, into shared memory (rows beyond the entry: zeros)
     for (int i = tid; i < M * ROWS * (D / 8); i += THREADS) {
@@ -224,14 +231,14 @@ mapped_attention_mma_kernel(const MmaParams p) {
         }
         if (!any) continue;
         // ---- S = Q K^T
-        float s[KT / 8][4];
+        float s[KW / 8][4];
 #pragma unroll
-        for (int j = 0; j < KT / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
-        const bf16* kt = Ks + ((size_t)buf * M + map) * KT * KP;
+        for (int j = 0; j < KW / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
+        const bf16* kt = Ks + (((size_t)buf * M + map) * KT + k_off) * KP;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {
 #pragma unroll
-            for (int jp = 0; jp < KT / 16; ++jp) {
+            for (int jp = 0; jp < KW / 16; ++jp) {
                 uint32_t b[4];
                 ldsm_x4(b, kt + ((size_t)jp * 16 + (lane & 7) + (lane >> 4) * 8) * KP + ks * 16 + ((lane >> 3) & 1) * 8);
                 mma_bf16(s[2 * jp], qf[ks], b[0], b[1]);
@@ -253,17 +260,18 @@ mapped_attention_mma_kernel(const MmaParams p) {
         const float sc2 = p.scale * LOG2E, inv_cap = p.softcap > 0.f ? p.scale / p.softcap : 0.f, cap2 = p.softcap * LOG2E;
         float mx_a = -INFINITY, mx_b = -INFINITY;
 #pragma unroll
-        for (int j = 0; j < KT / 8; ++j) {
+        for (int j = 0; j < KW / 8; ++j) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
+                const int kc = k_off + j * 8 + 2 * tq + (e & 1);               // the key's column in the tile
                 float v = p.softcap > 0.f ? cap2 * tanh_ex2(s[j][e] * inv_cap) : s[j][e] * sc2;
                 const int pos = (e < 2) ? pos_a : pos_b;
                 if (p.slopes) {
-                    const int kp = interior ? tile_first + j * 8 + 2 * tq + (e & 1) : kpos_t[j * 8 + 2 * tq + (e & 1)];
+                    const int kp = interior ? tile_first + kc : kpos_t[kc];
                     v -= ((e < 2) ? slope_a : slope_b) * (float)(pos - kp);
                 }
                 if (!interior) {
-                    const int kpos = kpos_t[j * 8 + 2 * tq + (e & 1)];
+                    const int kpos = kpos_t[kc];
                     const bool row_ok = ((e < 2) ? row_a : row_b) < n_rows;
                     const bool vis = row_ok && kpos >= ((e < 2) ? cs_a : cs_b) && kpos <= pos &&
                                      (p.window <= 0 || pos - kpos < p.window || kpos < p.keep_first);
@@ -285,7 +293,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
 #pragma unroll
         for (int j = 0; j < DV / 8; ++j) { o[j][0] *= ca; o[j][1] *= ca; o[j][2] *= cb; o[j][3] *= cb; }
 #pragma unroll
-        for (int j = 0; j < KT / 8; ++j) {
+        for (int j = 0; j < KW / 8; ++j) {
             s[j][0] = ex2f(s[j][0] - ua); s[j][1] = ex2f(s[j][1] - ua);        // 2^-inf = 0 for what the mask hides
             s[j][2] = ex2f(s[j][2] - ub); s[j][3] = ex2f(s[j][3] - ub);
             l_a += s[j][0] + s[j][1];
@@ -293,22 +301,30 @@ mapped_attention_mma_kernel(const MmaParams p) {
         }
         // ---- O += P V, P as three bfloat16 terms
 #pragma unroll
-        for (int kk = 0; kk < KT / 16; ++kk) {
+        for (int kk = 0; kk < KW / 16; ++kk) {
             uint32_t ah[4], am[4], al[4];
             split3(s[2 * kk][0], s[2 * kk][1], ah[0], am[0], al[0]);
             split3(s[2 * kk][2], s[2 * kk][3], ah[1], am[1], al[1]);
             split3(s[2 * kk + 1][0], s[2 * kk + 1][1], ah[2], am[2], al[2]);
             split3(s[2 * kk + 1][2], s[2 * kk + 1][3], ah[3], am[3], al[3]);
+            // a few groups of value columns take turns, so that the products of one accumulator are apart
+            const bf16* vt = Vs + (size_t)buf * KT * VP + ((size_t)k_off + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + (lane >> 4) * 8;
 #pragma unroll
-            for (int np = 0; np < DV / 16; ++np) {
-                uint32_t b[4];
-                ldsm_x4_t(b, Vs + (size_t)buf * KT * VP + ((size_t)kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VP + np * 16 + (lane >> 4) * 8);
-                mma_bf16(o[2 * np], al, b[0], b[1]);        // smallest terms first
-                mma_bf16(o[2 * np + 1], al, b[2], b[3]);
-                mma_bf16(o[2 * np], am, b[0], b[1]);
-                mma_bf16(o[2 * np + 1], am, b[2], b[3]);
-                mma_bf16(o[2 * np], ah, b[0], b[1]);
-                mma_bf16(o[2 * np + 1], ah, b[2], b[3]);
+            for (int n0 = 0; n0 < DV / 16; n0 += TURNS) {
+                uint32_t b[TURNS][4];
+#pragma unroll
+                for (int x = 0; x < TURNS; ++x)
+                    if (n0 + x < DV / 16) ldsm_x4_t(b[x], vt + (n0 + x) * 16);
+#pragma unroll
+                for (int term = 0; term < 3; ++term) {      // smallest terms first
+                    const uint32_t (&a)[4] = term == 0 ? al : term == 1 ? am : ah;
+#pragma unroll
+                    for (int x = 0; x < TURNS; ++x)
+                        if (n0 + x < DV / 16) {
+                            mma_bf16(o[2 * (n0 + x)], a, b[x][0], b[x][1]);
+                            mma_bf16(o[2 * (n0 + x) + 1], a, b[x][2], b[x][3]);
+                        }
+                }
             }
         }
     }
@@ -320,22 +336,37 @@ mapped_attention_mma_kernel(const MmaParams p) {
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 1);
     l_b += __shfl_xor_sync(0xffffffffu, l_b, 2);
     if (GROUP) {
-        // the run's state per head and map, as the kernel that merges runs reads it: maximum (natural logarithm), sum,
-        // weighted values relative to that maximum
-        if (warp_live) {
-            constexpr float LN2 = 0.6931471805599453f;
+        // the warps' states through shared memory, over the tiles; then, per head and map, their sum in warp order as the
+        // kernel that merges runs reads it: maximum (natural logarithm), sum, weighted values relative to that maximum
+        if (tq == 0) {
+            part_m[warp][gq] = m_a; part_m[warp][gq + 8] = m_b;
+            part_l[warp][gq] = l_a; part_l[warp][gq + 8] = l_b;
+        }
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int r = half ? row_b : row_a;
-                if (r < n_rows) {
-                    float* ps = p.partial + ((((size_t)q0 * p.nH + head + r) * p.n_splits + blockIdx.x) * M + map) * (DV + 2);
-                    if (tq == 0) { ps[0] = (half ? m_b : m_a) * LN2; ps[1] = half ? l_b : l_a; }
+        for (int j = 0; j < DV / 8; ++j) {
+            *reinterpret_cast<float2*>(Os + ((size_t)warp * 16 + gq) * DV + j * 8 + 2 * tq) = make_float2(o[j][0], o[j][1]);
+            *reinterpret_cast<float2*>(Os + ((size_t)warp * 16 + gq + 8) * DV + j * 8 + 2 * tq) = make_float2(o[j][2], o[j][3]);
+        }
+        __syncthreads();
+        constexpr float LN2 = 0.6931471805599453f;
+        for (int rm = warp; rm < n_rows * M; rm += WARPS) {
+            const int r = rm / M, m = rm % M;            // (the warps of map m are m, m + M, ...)
+            float mt = -INFINITY, f[PARTS], lt = 0.f;
 #pragma unroll
-                    for (int j = 0; j < DV / 8; ++j) {
-                        ps[2 + j * 8 + 2 * tq] = o[j][2 * half];
-                        ps[2 + j * 8 + 2 * tq + 1] = o[j][2 * half + 1];
-                    }
-                }
+            for (int x = 0; x < PARTS; ++x) mt = fmaxf(mt, part_m[m + x * M][r]);
+#pragma unroll
+            for (int x = 0; x < PARTS; ++x) {
+                const float mx = part_m[m + x * M][r];
+                f[x] = mx == -INFINITY ? 0.f : ex2f(mx - mt);
+                lt += part_l[m + x * M][r] * f[x];
+            }
+            float* ps = p.partial + ((((size_t)q0 * p.nH + head + r) * p.n_splits + blockIdx.x) * M + m) * (DV + 2);
+            if (lane == 0) { ps[0] = mt * LN2; ps[1] = lt; }
+            for (int c = lane; c < DV; c += 32) {
+                float a = 0.f;
+#pragma unroll
+                for (int x = 0; x < PARTS; ++x) a = fmaf(Os[((size_t)(m + x * M) * 16 + r) * DV + c], f[x], a);
+                ps[2 + c] = a;
             }
         }
         return;
@@ -367,8 +398,8 @@ mapped_attention_mma_kernel(const MmaParams p) {
                 ss += v[u] * v[u];
             }
         }
-        float r = 1.f;
-        if (p.head_norm) r = rsqrtf(ng_warp_sum(ss) / (float)DV + p.eps) * p.post_scale;
+        float r = p.post_scale;
+        if (p.head_norm) r *= rsqrtf(ng_warp_sum(ss) / (float)DV + p.eps);
         bf16* dst = p.out + (size_t)(q0 + r0 + row) * p.out_ld + (size_t)head * DV;
 #pragma unroll
         for (int u = 0; u < DV / 32 + 1; ++u) {
@@ -382,7 +413,7 @@ template <int M, bool GROUP>
 static int mma_launch(const MmaParams& p, int n_entries, int max_q, cudaStream_t stream) {
     constexpr int ROWS = (WARPS / M) * 16;
     const size_t tiles = ((size_t)M * ROWS * QP + 2 * ((size_t)M * KT * KP + (size_t)KT * VP)) * sizeof(bf16);
-    const size_t epi = (size_t)M * ROWS * QP * sizeof(bf16) + (size_t)M * ROWS * DV * sizeof(float);
+    const size_t epi = (size_t)M * ROWS * QP * sizeof(bf16) + (size_t)(M * ROWS > 64 ? M * ROWS : 64) * DV * sizeof(float);
     const size_t smem = tiles > epi ? tiles : epi;
     static bool attr = false;
     if (!attr) {

@@ -448,16 +448,22 @@ def mapped_attention_partial_floats(n_rows: int, n_heads: int, n_maps: int, vdim
     return n_rows * n_heads * n_splits * n_maps * (vdim + 2) if n_splits > 1 else 0
 
 
+def _post(head_norm: bool, post_scale: float, out_scale: float) -> float:
+    """What the kernels multiply a finished head by."""
+    return float(post_scale if head_norm else 1.0) * float(out_scale)
+
+
 def mapped_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, table: torch.Tensor,
                      positions: torch.Tensor, row_entry: torch.Tensor, out: torch.Tensor, n_heads: int, n_maps: int,
                      window: Optional[int], keep_first: int, scale: float, softcap: float, lam: float, head_norm: bool,
                      post_scale: float, eps: float, n_splits: int = 1, partial: Optional[torch.Tensor] = None,
-                     slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
+                     slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
+                     out_scale: float = 1.0) -> None:
     """Attention with float32 scores and weights over keys [P, G * n_maps, page, dim] and values [P, G, page, vdim]:
     per head and map m, a_m = softmax(cap(scale * q_m . k_m)) v over the keys j <= pos with pos - j < window or
     j < keep_first (window None: all), cap(s) = softcap * tanh(s / softcap) (softcap 0: none); the head's output is
     a_0 (one map) or a_0 - lam * a_1 (two), then, with ``head_norm``, over its root mean square (eps) times
-    ``post_scale``.  ``out`` [N, n_heads * vdim] may be a block of columns of a wider buffer.  ``n_splits`` > 1 cuts
+    ``post_scale``; times ``out_scale`` in any case.  ``out`` [N, n_heads * vdim] may be a block of columns of a wider buffer.  ``n_splits`` > 1 cuts
     every row's keys into runs, a block each, merged through ``partial`` (float32,
     ``mapped_attention_partial_floats`` values): for steps of few rows.  ``slopes`` (float32 [n_heads]): slope[head] *
     (position - key position) is taken off every score; ``sinks`` (float32 [n_heads]): every softmax's denominator
@@ -479,7 +485,7 @@ def mapped_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     _check(f(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], _ptr(positions), _ptr(row_entry),
              out.data_ptr(), _column_block(out, "attention out"), _ptr(partial) if need else None, n, n_heads, n_g, n_maps,
              dim, vdim, page_size, num_pages, int(window or 0), int(keep_first), int(n_splits), float(scale),
-             float(softcap or 0.0), float(lam), float(post_scale), float(eps), int(bool(head_norm)),
+             float(softcap or 0.0), float(lam), _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)),
              _slopes(slopes, n_heads), _slopes(sinks, n_heads), int(chunk or 0), _act_flag(q, "q"), _stream()), "mapped_attention")
 
 
@@ -496,7 +502,8 @@ def mapped_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
                          cu_q: torch.Tensor, ctx_before: torch.Tensor, out: torch.Tensor, n_entries: int, max_q: int,
                          n_heads: int, n_maps: int, window: Optional[int], keep_first: int, scale: float, softcap: float,
                          lam: float, head_norm: bool, post_scale: float, eps: float,
-                         slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
+                         slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
+                     out_scale: float = 1.0) -> None:
     """``mapped_attention`` for long bfloat16 steps on the tensor cores: scores are float32 sums of exact bfloat16
     products, the float32 softmax weights enter the weighted sum as three bfloat16 terms each.  Rows are named by
     ``cu_q`` [R+1] and ``ctx_before`` [R]; ``max_q`` bounds the longest entry."""
@@ -513,7 +520,7 @@ def mapped_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
     _check(f(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], _ptr(cu_q), _ptr(ctx_before),
              out.data_ptr(), _column_block(out, "attention out"), n_entries, max_q, n_heads, n_g, n_maps, dim, vdim,
              page_size, num_pages, int(window or 0), int(keep_first), float(scale), float(softcap or 0.0), float(lam),
-             float(post_scale), float(eps), int(bool(head_norm)), _slopes(slopes, n_heads), _slopes(sinks, n_heads),
+             _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)), _slopes(slopes, n_heads), _slopes(sinks, n_heads),
              int(chunk or 0), _stream()), "mapped_attention_mma")
 
 
@@ -527,7 +534,7 @@ def mapped_attention_group(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
                            partial: torch.Tensor, n_entries: int, n_heads: int, n_maps: int, window: Optional[int],
                            keep_first: int, scale: float, softcap: float, lam: float, head_norm: bool, post_scale: float,
                            eps: float, n_splits: int, slopes: Optional[torch.Tensor] = None,
-                           sinks: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
+                           sinks: Optional[torch.Tensor] = None, chunk: int = 0, out_scale: float = 1.0) -> None:
     """``mapped_attention`` for a step whose entries bring one token each (bfloat16), on the tensor cores: the query
     heads of a KV group are the rows of a tile, every row's keys are cut into ``n_splits`` runs (a block each), and the
     runs' states pass through ``partial`` (float32, ``mapped_attention_partial_floats`` values, also for one run) to
@@ -552,7 +559,7 @@ def mapped_attention_group(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
     g = _fn("mapped_attention", "ng_mapped_attention_merge", [_c_void_p] * 3 + [_c_int] * 6 + [_c_float] * 3
             + [_c_int, _c_void_p, _c_int, _c_void_p])
     _check(g(_ptr(partial), _ptr(row_entry), out.data_ptr(), _column_block(out, "attention out"), n, n_heads, n_maps, vdim,
-             int(n_splits), float(lam), float(post_scale), float(eps), int(bool(head_norm)), _slopes(sinks, n_heads), 1, _stream()),
+             int(n_splits), float(lam), _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)), _slopes(sinks, n_heads), 1, _stream()),
            "mapped_attention_merge")
 
 
@@ -993,6 +1000,12 @@ def decayed_linear_scratch(n_rows: int, n_entries: int, n_heads: int, key_dim: i
     return slots * n_heads * (key_dim * value_dim + key_dim + 2) + n_rows * n_heads * 4 + 8
 
 
+def decay_powers(decay, device) -> torch.Tensor:
+    """float32 [nH, DECAYED_CHUNK + 1]: every head's decay to the powers 0 .. DECAYED_CHUNK, formed in float64."""
+    base = torch.as_tensor(decay, dtype=torch.float64).reshape(-1, 1)
+    return base.pow(torch.arange(DECAYED_CHUNK + 1, dtype=torch.float64)).to(torch.float32).to(device).contiguous()
+
+
 def _decayed_linear(what, x, gates, gate_bias, decay, cap, state, nm_state, o_raw, norm_w, out, cu_q, ctx_before, slots,
                     row_entry, n_entries, n_heads, key_dim, value_dim, norm_group, eps, out_scale, scratch, max_q):
     n = x.shape[0]
@@ -1028,13 +1041,14 @@ def lightning(x: torch.Tensor, decay: torch.Tensor, norm_w: torch.Tensor, state:
               out: torch.Tensor, cu_q: torch.Tensor, ctx_before: torch.Tensor, slots: torch.Tensor, row_entry: torch.Tensor,
               n_entries: int, n_heads: int, key_dim: int, value_dim: int, eps: float, out_scale: float = 1.0,
               scratch: Optional[torch.Tensor] = None, max_q: int = 0) -> None:
-    """x[N, 2*nH*(dk+dv)] = q|k|v|g;  q, k, v <- silu (rounded to x's dtype);  per head S = decay*S + k v^T, o = S^T q;
+    """x[N, 2*nH*(dk+dv)] = q|k|v|g;  q, k, v <- silu (rounded to x's dtype);  per head S = decay*S + k v^T, o = S^T q
+    (``decay`` [nH, DECAYED_CHUNK + 1]: the decays' powers, ``decay_powers``);
     out[N, nH*dv] = o / rms(o over all heads together) * norm_w * sigmoid(g) * out_scale;  state[slots, nH, dk, dv] and
     the scratch ``o_raw`` [N, nH*dv] float32.  ``out`` may be a block of columns of a wider buffer.  With ``scratch``
     (``decayed_linear_scratch`` float32 values) and ``max_q`` (the longest portion) the chunk-by-chunk tensor-core
     kernels run (bfloat16; ``decayed_linear_chunked_takes``); else the token-by-token kernel."""
-    if decay.numel() != n_heads:
-        raise KernelError("lightning: a decay per head")
+    if decay.shape != (n_heads, DECAYED_CHUNK + 1):
+        raise KernelError("lightning: the powers of a decay per head (decay_powers)")
     _decayed_linear("lightning", x, None, None, decay, 0.0, state, None, o_raw, norm_w, out, cu_q, ctx_before, slots, row_entry,
                     n_entries, n_heads, key_dim, value_dim, n_heads * value_dim, eps, out_scale, scratch, max_q)
 

@@ -86,7 +86,7 @@ class LightningAttention(_DecayedLinear):
 
     def __init__(self, spec, *, dtype, device):
         super().__init__(spec, dtype=dtype, device=device)
-        self.decay = torch.tensor(spec.decay, dtype=torch.float64).to(torch.float32).to(device)
+        self.decay = ops.decay_powers(spec.decay, device)
 
     def cache_need(self):
         s = self.spec

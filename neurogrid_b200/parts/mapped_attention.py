@@ -173,16 +173,16 @@ class MappedAttention:
                      half_pairing=bool(pa.inv_freq is not None and pa.half_pairing),
                      unit_norm=bool(s.qk_norm and not getattr(s, "norm_weight", True)),
                      v_is_k=bool(self.shared_kv and n_v), rot_mag=pa.magnitude if pa.inv_freq is not None else 1.0)
-        self.attend(q, cache, ctx, out, pa.score_slopes)
-        if gated or out_scale != 1.0:
+        self.attend(q, cache, ctx, out, pa.score_slopes, 1.0 if gated else out_scale)
+        if gated:
             ops.gate_mul(out, gate, "sigmoid", out_scale)
 
-    def attend(self, q, cache, ctx, out, slopes=None):
+    def attend(self, q, cache, ctx, out, slopes=None, out_scale=1.0):
         """The attention core over the pages: q [N, n_heads * n_maps * key_dim] as the preparation left it.
         ``slopes``: the position encoding's score bias per head, if it has one."""
         s = self.spec
         n = q.shape[0]
-        extra = dict(slopes=slopes, sinks=self.sinks, chunk=getattr(s, "chunk", None) or 0)
+        extra = dict(slopes=slopes, sinks=self.sinks, chunk=getattr(s, "chunk", None) or 0, out_scale=out_scale)
         if ctx.max_q == 1 and n <= self.GROUP_MAX_ROWS and not ctx.fixed_launches and \
                 ops.mapped_attention_group_takes(s.key_dim, s.value_dim, s.n_heads, s.n_kv_heads, self.dtype):
             n_splits = self._group_splits(n, cache)

@@ -140,7 +140,8 @@ def qkv_prep(qkv, q_out, q_weight, k_weight, inv_freq, k_pages, v_pages, table, 
 
 
 def mapped_attention(q, k_pages, v_pages, table, positions, row_entry, out, n_heads, n_maps, window, keep_first, scale,
-                     softcap, lam, head_norm, post_scale, eps, n_splits=1, partial=None, slopes=None, sinks=None, chunk=0):
+                     softcap, lam, head_norm, post_scale, eps, n_splits=1, partial=None, slopes=None, sinks=None, chunk=0,
+                     out_scale=1.0):
     n = q.shape[0]
     P, n_k, ps, dim = k_pages.shape
     n_g, vdim = v_pages.shape[1], v_pages.shape[3]
@@ -177,7 +178,7 @@ def mapped_attention(q, k_pages, v_pages, table, positions, row_entry, out, n_he
             y = a[0] if n_maps == 1 else a[0] - lam * a[1]
             if head_norm:
                 y = y * torch.rsqrt((y * y).mean() + eps) * post_scale
-            o[h] = y
+            o[h] = y * out_scale
         out[r] = o.reshape(-1).to(out.dtype)
 
 
@@ -508,6 +509,7 @@ def _norm_gate(o, group, norm_w, gate, eps, out_scale):
 def lightning(x, decay, norm_w, state, o_raw, out, cu_q, ctx_before, slots, row_entry, n_entries, n_heads, key_dim, value_dim,
               eps, out_scale=1.0, scratch=None, max_q=0):
     H, dk, dv = n_heads, key_dim, value_dim
+    decay = decay[:, 1]
     act = lambda t: (t * torch.sigmoid(t)).to(x.dtype).to(D)              # rounded to the activation type
     for e in range(n_entries):
         r0, r1 = int(cu_q[e]), int(cu_q[e + 1])

@@ -169,20 +169,23 @@ def test_keys_as_values_and_a_rescaled_rotation(dtype, n_q, n_k, dim, rot, extra
     assert int(ctx.status.item()) == 0
 
 
-def _attend(kind, q, kp, vp, table, ctx, H, scale, sinks, n_splits=1):
+def _attend(kind, q, kp, vp, table, ctx, H, scale, sinks, n_splits=1, out_scale=0.6):
+    """Every head times ``out_scale`` in the kernel; taken out again here."""
     n, vdim = q.shape[0], vp.shape[3]
     out = torch.empty(n, H * vdim, dtype=q.dtype, device=DEV)
     args = (H, 1, None, 0, scale, 0.0, 0.0, False, 1.0, 1e-6)
     if kind == "rows":
         partial = torch.empty(max(1, ops().mapped_attention_partial_floats(n, H, 1, vdim, n_splits)), device=DEV) if n_splits > 1 else None
-        ops().mapped_attention(q, kp, vp, table, ctx.positions, ctx.row_entry, out, *args, n_splits, partial, sinks=sinks)
+        ops().mapped_attention(q, kp, vp, table, ctx.positions, ctx.row_entry, out, *args, n_splits, partial, sinks=sinks,
+                               out_scale=out_scale)
     elif kind == "tiles":
-        ops().mapped_attention_mma(q, kp, vp, table, ctx.cu_q, ctx.ctx_before, out, ctx.n_entries, ctx.max_q, *args, sinks=sinks)
+        ops().mapped_attention_mma(q, kp, vp, table, ctx.cu_q, ctx.ctx_before, out, ctx.n_entries, ctx.max_q, *args, sinks=sinks,
+                                   out_scale=out_scale)
     else:
         partial = torch.empty(n * H * n_splits * (vdim + 2), device=DEV)
         ops().mapped_attention_group(q, kp, vp, table, ctx.cu_q, ctx.ctx_before, ctx.row_entry, out, partial, ctx.n_entries, *args,
-                                     n_splits, sinks=sinks)
-    return out
+                                     n_splits, sinks=sinks, out_scale=out_scale)
+    return out.double() / out_scale
 
 
 def _plain_attend(q, k, v, H, scale, rows):
@@ -243,8 +246,7 @@ def _lightning_inputs(dtype, T, H, dk, dv, seed=0):
     g = torch.Generator().manual_seed(seed)
     rnd = lambda t: t.to(torch.bfloat16).to(dtype).to(DEV)
     x = rnd(1.5 * torch.randn(T, 2 * H * (dk + dv), generator=g))
-    decay = torch.tensor([0.97, 0.0, 1.0, 0.4, 0.999, 0.8][:H], device=DEV)
-    return x, decay, (1 + 0.2 * torch.randn(H * dv, generator=g)).to(DEV)
+    return x, [0.97, 0.0, 1.0, 0.4, 0.999, 0.8][:H], (1 + 0.2 * torch.randn(H * dv, generator=g)).to(DEV)
 
 
 def _mlstm_inputs(dtype, T, H, dk, dv, seed=0):
@@ -265,7 +267,7 @@ class _Recurrence:
     def __init__(self, kind, dtype, T, H, dk, dv, seed=0, cap=6.0):
         self.kind, self.dtype, self.H, self.dk, self.dv, self.cap = kind, dtype, H, dk, dv, cap
         if kind == "lightning":
-            self.x, self.decay, self.nw = _lightning_inputs(dtype, T, H, dk, dv, seed)
+            self.x, self.decay, self.nw = _lightning_inputs(dtype, T, H, dk, dv, seed)      # (a decay per head)
         else:
             self.x, self.gates, self.bias, self.nw = _mlstm_inputs(dtype, T, H, dk, dv, seed)
 
@@ -287,7 +289,7 @@ class _Recurrence:
                                          device=DEV), max_q=max(ctx.q_lens))
         tail = (out, ctx.cu_q, ctx.ctx_before, ctx.slots, ctx.row_entry, ctx.n_entries, self.H, self.dk, self.dv, 1e-5, scale)
         if self.kind == "lightning":
-            ops().lightning(x, self.decay, self.nw, states[0], raw, *tail, **kw)
+            ops().lightning(x, ops().decay_powers(self.decay, DEV), self.nw, states[0], raw, *tail, **kw)
         else:
             ops().mlstm(x, self.gates[rows].contiguous(), self.bias, self.cap, self.nw, states[0], states[1], raw, *tail, **kw)
 
@@ -299,7 +301,7 @@ class _Recurrence:
         v, g = x[:, 2 * H * dk:2 * H * dk + H * dv].view(-1, H, dv), x[:, 2 * H * dk + H * dv:]
         if self.kind == "lightning":
             act = lambda t: plain.silu(t).to(self.dtype).double()
-            o, S = plain.decayed_sum(act(q), act(k), act(v), self.decay.double().cpu(), None if states is None else states[0])
+            o, S = plain.decayed_sum(act(q), act(k), act(v), self.decay, None if states is None else states[0])
             o, new = plain.rms_norm(o.reshape(-1, H * dv), self.nw.double().cpu(), 1e-5), (S,)
         else:
             pre = self.cap * torch.tanh((self.gates[rows].double().cpu() + self.bias.double().cpu()) / self.cap)
@@ -414,7 +416,7 @@ def test_a_key_far_back_shows(kind, chunked):
     r.x[far, 2 * dk:2 * dk + dv] = torch.linspace(-4, 4, dv).to(DEV)
     r.x[far + 700, :dk] = r.x[far, dk:2 * dk]
     if kind == "lightning":
-        r.decay[:] = 0.9995
+        r.decay = [0.9995]
     else:
         r.gates[:, :H], r.gates[:, H:], r.bias[:] = -2.0, 9.0, 0.0
         r.gates[far, 0] = 5.0
