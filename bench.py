@@ -1462,7 +1462,7 @@ def matepel_kernel_times(eng, l2, pk):
                 nm = torch.zeros(8, nH, ops.decayed_linear_slices(dv), dk + 1, device=dev)
                 run = lambda: ops.mlstm(p, gates, part.b_gates, spec.gate_cap, part.norm, state, nm, *tail, **kw)
                 xs = rnd(rows, D)
-                mem(f"{tag}_mlstm_gate_product", timed(lambda: ops.linear(xs, part.w_gates, None, gates)),
+                mem(f"{tag}_mlstm_gate_product", timed(lambda: ops.linear_f32(xs, part.w_gates, ctx.ws, "gates")),
                     rows * D * 2 + part.w_gates.numel() * 2 + gates.numel() * 4)
             else:
                 run = lambda: ops.lightning(p, part.decay, part.norm, state, *tail, **kw)

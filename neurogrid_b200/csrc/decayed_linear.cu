@@ -48,6 +48,8 @@ enum { DL_LIGHTNING = 0, DL_MLSTM = 1 };
 
 struct DlGeom {
     int nH, dk, dv;
+    int g_parts;               // mLSTM: float32 partial sums the gates' preactivations come as (1: whole)
+    size_t g_stride;           // ... elements between them
 };
 
 __device__ __forceinline__ float dl_silu(float z) { return z / (1.f + expf(-z)); }
@@ -62,7 +64,15 @@ __device__ __forceinline__ float dl_silu_as(float z) {
     return ng_ld(&r);
 }
 __device__ __forceinline__ float dl_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
-__device__ __forceinline__ void dl_log_gates(float xi, float xf, float bi, float bf, float cap, float& li, float& lf) {
+// the log gates of one row and head; `gr`: the row's preactivations i | f, or n_part partial sums of them, `stride` apart
+__device__ __forceinline__ void dl_log_gates(const float* gr, int head, int nH, int n_part, size_t stride, float bi, float bf,
+                                             float cap, float& li, float& lf) {
+    float xi = 0.f, xf = 0.f;
+#pragma unroll 4
+    for (int s = 0; s < n_part; ++s) {
+        xi += gr[s * stride + head];
+        xf += gr[s * stride + nH + head];
+    }
     li = cap * tanhf((xi + bi) / cap);
     lf = dl_log_sigmoid(cap * tanhf((xf + bf) / cap));
 }
@@ -136,7 +146,7 @@ dl_step_kernel(const T* __restrict__ x, const float* __restrict__ gates, const f
             float li = 0.f, lf = 0.f;
             if (lane < nt) {
                 const float* gr = gt + (size_t)(q0 + t0 + lane) * 2 * nH;
-                dl_log_gates(gr[head], gr[nH + head], gate_bias[head], gate_bias[nH + head], cap, li, lf);
+                dl_log_gates(gr, head, nH, geo.g_parts, geo.g_stride, gate_bias[head], gate_bias[nH + head], cap, li, lf);
             }
             float mm = m, keep = 0.f, add = 0.f, em = 0.f;
             for (int t = 0; t < nt; ++t) {
@@ -368,7 +378,8 @@ __device__ __forceinline__ void dl_load_tile(bf16* dst, int pitch, const bf16* _
 __global__ void __launch_bounds__(1024)
 dl_gates_kernel(const float* __restrict__ gates, const float* __restrict__ gate_bias, float cap, float4* __restrict__ tok,
                 float2* __restrict__ chk, float* __restrict__ nm_state, const int* __restrict__ cu_q,
-                const int* __restrict__ ctx_before, const int* __restrict__ slots, int nH, int dk, int slices) {
+                const int* __restrict__ ctx_before, const int* __restrict__ slots, DlGeom geo, int slices) {
+    const int nH = geo.nH, dk = geo.dk;
     __shared__ float sum_s[32], top_s[32], m_s[33];
     ng_pdl_trigger();
     ng_pdl_wait();
@@ -389,7 +400,7 @@ dl_gates_kernel(const float* __restrict__ gates, const float* __restrict__ gate_
             lf[u] = 0.f;
             if (tb + u < qlen) {
                 const float* gr = gates + (size_t)(q0 + tb + u) * 2 * nH;
-                dl_log_gates(gr[head], gr[nH + head], bi, bf, cap, li[u], lf[u]);
+                dl_log_gates(gr, head, nH, geo.g_parts, geo.g_stride, bi, bf, cap, li[u], lf[u]);
             }
         }
         // F of the lane's two tokens: a scan of the pairs' sums
@@ -750,15 +761,17 @@ static int dl_step(const void* x, const float* gates, const float* gate_bias, co
 
 // Token by token.  x [n_rows, 2 nH (dk + dv)]; lightning (gates null): decay [nH][DC + 1], the powers of every head's
 // decay; mLSTM: gates [n_rows, 2 nH] float32
-// preactivations i | f, gate_bias [2 nH], nm_state [slots, nH, ng_dl_slices(dv), dk + 1].  o_raw float32 [n_rows, nH dv].
+// preactivations i | f, or g_parts partial sums of them g_stride elements apart, gate_bias [2 nH], nm_state [slots, nH, ng_dl_slices(dv), dk + 1].  o_raw float32 [n_rows, nH dv].
 NG_EXPORT int ng_dl_step(const void* x, const float* gates, const float* gate_bias, const float* decay, float cap,
                          float* state, float* nm_state, float* o_raw, const int* cu_q, const int* ctx_before,
-                         const int* slots, int n_entries, int nH, int dk, int dv, int act_bf16, cudaStream_t stream) {
+                         const int* slots, int n_entries, int nH, int dk, int dv, int g_parts, long long g_stride,
+                         int act_bf16, cudaStream_t stream) {
     if (n_entries <= 0) return NG_OK;
+    if (g_parts < 1) return NG_BAD_SIZE;
     if (nH <= 0 || nH > 65535 || dk <= 0 || dk > DL_ROWS * DL_MAX_WARPS || dv <= 0 || ng_dl_slices(dv) > 65535 || !state || !o_raw)
         return NG_BAD_SIZE;
     if (gates ? (!gate_bias || !nm_state || !(cap > 0.f)) : !decay) return NG_BAD_SIZE;
-    const DlGeom geo{nH, dk, dv};
+    const DlGeom geo{nH, dk, dv, g_parts, (size_t)g_stride};
 #define DL_STEP(TT, MM) dl_step<TT, MM>(x, gates, gate_bias, decay, cap, state, nm_state, o_raw, cu_q, ctx_before, slots, n_entries, geo, stream)
     if (act_bf16) return gates ? DL_STEP(bf16, DL_MLSTM) : DL_STEP(bf16, DL_LIGHTNING);
     return gates ? DL_STEP(float, DL_MLSTM) : DL_STEP(float, DL_LIGHTNING);
@@ -795,7 +808,7 @@ static int dl_chunked(const bf16* x, const float* gates, const float* gate_bias,
     if (grid.y > 65535 || grid.z > 65535 || so > 200 * 1024) return NG_BAD_SIZE;
     if (MODE == DL_MLSTM)
         NG_LAUNCH((dl_gates_kernel), dim3(n_entries, geo.nH), 1024, 0, stream, gates, gate_bias, cap, tok, chk, nm, cu_q, ctx, slots,
-                  geo.nH, geo.dk, step_slices);
+                  geo, step_slices);
     NG_LAUNCH((dl_local_kernel<MODE, DVS>), grid, DC_THREADS, sl, stream, x, (const float4*)tok, decay, u, un, cu_q, geo);
     NG_LAUNCH((dl_scan_kernel<MODE>), sgrid, 256, 0, stream, u, un, state, nm, decay, (const float2*)chk, cu_q, ctx, slots, geo, step_slices);
     NG_LAUNCH((dl_out_kernel<MODE, DVS>), grid, DC_THREADS, so, stream, x, (const float4*)tok, (const float2*)chk, decay,
@@ -808,13 +821,14 @@ static int dl_chunked(const bf16* x, const float* gates, const float* gate_bias,
 NG_EXPORT int ng_dl_chunked(const void* x, const float* gates, const float* gate_bias, const float* decay, float cap,
                             float* state, float* nm_state, float* o_raw, float* scratch, const int* cu_q,
                             const int* ctx_before, const int* slots, int n_entries, int n_rows, int max_q, int nH, int dk,
-                            int dv, cudaStream_t stream) {
+                            int dv, int g_parts, long long g_stride, cudaStream_t stream) {
     if (n_entries <= 0 || n_rows <= 0 || max_q <= 0) return NG_OK;
+    if (g_parts < 1) return NG_BAD_SIZE;
     if (nH <= 0 || !ng_dl_chunked_takes(dk, dv) || !state || !o_raw || !scratch || ((uintptr_t)scratch & 15) ||
         ((uintptr_t)x & 15) || ((uintptr_t)state & 15) || ((uintptr_t)o_raw & 7))
         return NG_BAD_SIZE;
     if (gates ? (!gate_bias || !nm_state || !(cap > 0.f)) : !decay) return NG_BAD_SIZE;
-    const DlGeom geo{nH, dk, dv};
+    const DlGeom geo{nH, dk, dv, g_parts, (size_t)g_stride};
     const int dvs = dv % 64 == 0 ? 64 : dv % 32 == 0 ? 32 : 16;
 #define DL_CHUNKED(MM, SS) dl_chunked<MM, SS>((const bf16*)x, gates, gate_bias, decay, cap, state, nm_state, o_raw, scratch, cu_q, \
                                               ctx_before, slots, n_entries, n_rows, max_q, geo, stream)

@@ -131,6 +131,104 @@ hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __
         for (int v = 0; v < VEC; ++v) ng_st(out + row * H + j + v, u_s[j + v] * r * norm_w[j + v]);
 }
 
+// four neighbouring values
+__device__ __forceinline__ float4 hc_ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 hc_ld4(const __nv_bfloat16* p) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xffff0000u), __uint_as_float(u.y << 16),
+                       __uint_as_float(u.y & 0xffff0000u));
+}
+__device__ __forceinline__ void hc_st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void hc_st4(__nv_bfloat16* p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+// The same for rows that a block holds at once, four columns a thread (H % 4 == 0, H <= 4 * blockDim): what does not
+// depend on the kernel before (mixing matrix, weights, bias) is read before the wait, the partial sums are fetched four
+// at a time, and the row's read-out stays in registers between its sum of squares and its norm.
+template <typename TD, typename TO, int S>
+__global__ void __launch_bounds__(512)
+hc_step_row_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __restrict__ delta, int n_partials,
+                   size_t partial_stride, const float* __restrict__ mix, const float* __restrict__ out_w,
+                   const float* __restrict__ in_w, const float* __restrict__ norm_w, TO* __restrict__ out,
+                   float* __restrict__ sum_out, const float* __restrict__ bias, int H, float eps) {
+    __shared__ float red[32];
+    __shared__ float mix_s[S * S], ow_s[S], iw_s[S];
+    ng_pdl_trigger();
+    const int j = threadIdx.x * 4;
+    const bool live = j < H;
+    for (int i = threadIdx.x; i < S * S; i += blockDim.x) mix_s[i] = delta ? mix[i] : 0.f;
+    if (threadIdx.x < S) {
+        ow_s[threadIdx.x] = delta ? out_w[threadIdx.x] : 0.f;
+        iw_s[threadIdx.x] = in_w ? in_w[threadIdx.x] : 0.f;
+    }
+    const float4 zero = make_float4(0.f, 0.f, 0.f, 0.f);
+    const float4 nw = in_w && live ? hc_ld4(norm_w + j) : zero;
+    float4 y = bias && live ? hc_ld4(bias + j) : zero;
+    __syncthreads();
+    ng_pdl_wait();
+    delta = ng_after_wait(delta);
+    x0 = ng_after_wait(x0);
+    const size_t row = blockIdx.x;
+    float* xr = X + row * (size_t)S * H + j;
+    float4 xs[S], u = zero;
+    if (live) {
+        if (x0) {
+            const float4 t = hc_ld4(x0 + row * H + j);
+#pragma unroll
+            for (int s = 0; s < S; ++s) xs[s] = t;
+        } else {
+#pragma unroll
+            for (int s = 0; s < S; ++s) xs[s] = hc_ld4(xr + (size_t)s * H);
+        }
+        if (delta) {
+            float4 a = zero;
+#pragma unroll 4
+            for (int p = 0; p < n_partials; ++p) {      // ascending p
+                const float4 t = hc_ld4(delta + p * partial_stride + row * H + j);
+                a.x += t.x; a.y += t.y; a.z += t.z; a.w += t.w;
+            }
+            y.x += a.x; y.y += a.y; y.z += a.z; y.w += a.w;
+            float4 nx[S];
+#pragma unroll
+            for (int t = 0; t < S; ++t) {
+                float4 v = zero;
+#pragma unroll
+                for (int s = 0; s < S; ++s) {
+                    const float m = mix_s[s * S + t];
+                    v.x = fmaf(m, xs[s].x, v.x); v.y = fmaf(m, xs[s].y, v.y); v.z = fmaf(m, xs[s].z, v.z); v.w = fmaf(m, xs[s].w, v.w);
+                }
+                const float w = ow_s[t];
+                nx[t] = make_float4(fmaf(w, y.x, v.x), fmaf(w, y.y, v.y), fmaf(w, y.z, v.z), fmaf(w, y.w, v.w));
+            }
+#pragma unroll
+            for (int t = 0; t < S; ++t) xs[t] = nx[t];
+        }
+        if (delta || x0) {
+#pragma unroll
+            for (int s = 0; s < S; ++s) hc_st4(xr + (size_t)s * H, xs[s]);
+        }
+        if (sum_out) {
+            float4 t = zero;
+#pragma unroll
+            for (int s = 0; s < S; ++s) { t.x += xs[s].x; t.y += xs[s].y; t.z += xs[s].z; t.w += xs[s].w; }
+            hc_st4(sum_out + row * H + j, t);
+        }
+        if (in_w) {
+#pragma unroll
+            for (int s = 0; s < S; ++s) {
+                const float w = iw_s[s];
+                u.x = fmaf(w, xs[s].x, u.x); u.y = fmaf(w, xs[s].y, u.y); u.z = fmaf(w, xs[s].z, u.z); u.w = fmaf(w, xs[s].w, u.w);
+            }
+        }
+    }
+    if (!in_w) return;
+    const float ss = ng_block_sum(u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w, red);
+    const float r = rsqrtf(ss / (float)H + eps);
+    if (live) hc_st4(out + row * H + j, make_float4(u.x * r * nw.x, u.y * r * nw.y, u.z * r * nw.z, u.w * r * nw.w));
+}
+
 template <typename TD, typename TO, int S_CT, int VEC>
 static int hc_launch(float* X, const float* x0, const void* delta, int n_partials, size_t ps, const float* mix,
                      const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
@@ -157,8 +255,17 @@ static int hc_by_streams(float* X, const float* x0, const void* delta, int n_par
                          const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
                          int H, float eps, cudaStream_t stream) {
     const bool vec = H % 4 == 0 && ((uintptr_t)X & 15) == 0;
+    // rows that a block holds at once: four columns a thread, at most 512 threads
+    const bool row_at_once = vec && H <= 2048 && ps % 4 == 0 && ((uintptr_t)delta % (4 * sizeof(TD))) == 0 &&
+                             ((uintptr_t)out % (4 * sizeof(TO))) == 0 &&
+                             (((uintptr_t)x0 | (uintptr_t)sum_out | (uintptr_t)norm_w | (uintptr_t)bias) & 15) == 0;
 #define HC_CASE(SS)                                                                                                    \
     case SS:                                                                                                           \
+        if (row_at_once) {                                                                                             \
+            NG_LAUNCH((hc_step_row_kernel<TD, TO, SS>), n_rows, (H / 4 + 31) / 32 * 32, 0, stream, X, x0, (const TD*)delta, \
+                      n_partials, ps, mix, out_w, in_w, norm_w, (TO*)out, sum_out, bias, H, eps);                      \
+            return ng_launch_status();                                                                                 \
+        }                                                                                                              \
         return vec ? hc_launch<TD, TO, SS, 4>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream) \
                    : hc_launch<TD, TO, SS, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
     switch (S) {

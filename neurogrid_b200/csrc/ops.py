@@ -1018,18 +1018,22 @@ def _decayed_linear(what, x, gates, gate_bias, decay, cap, state, nm_state, o_ra
         _f32(t, w)
     _i32(cu_q, "cu_q"), _i32(ctx_before, "ctx_before"), _i32(slots, "slots"), _i32(row_entry, "row_entry")
     act = _act_flag(x, f"{what} input")
+    g_parts, g_stride = 1, 0
+    if gates is not None:
+        g_parts, g_stride = _stack(gates, (n, 2 * n_heads), torch.float32, f"{what} gates")
     common = (_ptr(x), _ptr(gates), _ptr(gate_bias), _ptr(decay), float(cap), _ptr(state), _ptr(nm_state), _ptr(o_raw))
     if scratch is not None:
         need = decayed_linear_scratch(n, n_entries, n_heads, key_dim, value_dim)
         if scratch.numel() < need or max_q <= 0 or x.dtype != torch.bfloat16 or not decayed_linear_chunked_takes(key_dim, value_dim):
             raise KernelError(f"{what}: the chunked kernels take bfloat16 and heads in sixteens, and need {need} float32 values "
                               "of scratch and the longest portion's length")
-        f = _fn("decayed_linear", "ng_dl_chunked", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 7 + [_c_int] * 6 + [_c_void_p])
+        f = _fn("decayed_linear", "ng_dl_chunked", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 7 + [_c_int] * 7 + [_c_ll, _c_void_p])
         _check(f(*common, _ptr(scratch), _ptr(cu_q), _ptr(ctx_before), _ptr(slots), n_entries, n, int(max_q), n_heads, key_dim,
-                 value_dim, _stream()), f"{what} (chunked)")
+                 value_dim, g_parts, g_stride, _stream()), f"{what} (chunked)")
     else:
-        f = _fn("decayed_linear", "ng_dl_step", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 6 + [_c_int] * 5 + [_c_void_p])
-        _check(f(*common, _ptr(cu_q), _ptr(ctx_before), _ptr(slots), n_entries, n_heads, key_dim, value_dim, act, _stream()), what)
+        f = _fn("decayed_linear", "ng_dl_step", [_c_void_p] * 4 + [_c_float] + [_c_void_p] * 6 + [_c_int] * 5 + [_c_ll, _c_int, _c_void_p])
+        _check(f(*common, _ptr(cu_q), _ptr(ctx_before), _ptr(slots), n_entries, n_heads, key_dim, value_dim, g_parts, g_stride,
+                 act, _stream()), what)
     gate_at = 2 * n_heads * key_dim + width                     # the output gate's columns of x
     f = _fn("decayed_linear", "ng_dl_finish", [_c_void_p] * 5 + [_c_int] * 5 + [_c_float, _c_float, _c_int, _c_void_p])
     _check(f(_ptr(o_raw), x.data_ptr() + gate_at * x.element_size(), _ptr(norm_w), out.data_ptr(), _ptr(row_entry), n, width,
@@ -1057,13 +1061,14 @@ def mlstm(x: torch.Tensor, gates: torch.Tensor, gate_bias: torch.Tensor, cap: fl
           state: torch.Tensor, nm_state: torch.Tensor, o_raw: torch.Tensor, out: torch.Tensor, cu_q: torch.Tensor,
           ctx_before: torch.Tensor, slots: torch.Tensor, row_entry: torch.Tensor, n_entries: int, n_heads: int, key_dim: int,
           value_dim: int, eps: float, out_scale: float = 1.0, scratch: Optional[torch.Tensor] = None, max_q: int = 0) -> None:
-    """x[N, 2*nH*(dk+dv)] = q|k|v|g and gates[N, 2*nH] float32 = preactivations i|f (``gate_bias`` [2*nH] is added here):
+    """x[N, 2*nH*(dk+dv)] = q|k|v|g and gates[N, 2*nH] float32 (or a stack [S, N, 2*nH] of partial sums) = preactivations
+    i|f (``gate_bias`` [2*nH] is added here):
     i = cap tanh(./cap), f = log sigmoid(cap tanh(./cap)), m' = max(f + m, i), S = exp(f + m - m') S + exp(i - m') k v^T,
     n likewise with k alone, o = s S^T q / (max(|s n.q|, exp(-m')) + 1e-6), s = dk^(-1/2);
     out[N, nH*dv] = o / rms(o of the head) * norm_w * sigmoid(g) * out_scale.  state[slots, nH, dk, dv] and
     nm_state[slots, nH, ``decayed_linear_slices(dv)``, dk+1] (n | m, one copy per slice) float32.  The rest as ``lightning``."""
     n = x.shape[0]
-    if gates.shape != (n, 2 * n_heads) or gate_bias.numel() != 2 * n_heads \
+    if gates.shape[-2:] != (n, 2 * n_heads) or gate_bias.numel() != 2 * n_heads \
             or nm_state.shape[1:] != (n_heads, decayed_linear_slices(value_dim), key_dim + 1):
         raise KernelError("mlstm: shapes do not fit")
     _decayed_linear("mlstm", x, gates, gate_bias, None, cap, state, nm_state, o_raw, norm_w, out, cu_q, ctx_before, slots,
@@ -1332,6 +1337,24 @@ def linear_to_residual(x: torch.Tensor, weight: torch.Tensor, bias: Optional[tor
             return buf
     out = ws.buf(name, M, N, x.dtype)
     linear(x, weight, bias, out)
+    return out
+
+
+def linear_f32(x: torch.Tensor, weight: torch.Tensor, ws, name: str):
+    """x @ weight^T in float32 for a consumer that adds partial sums: [M,N], or for few rows on the tcgen05 path a stack
+    [S,M,N] over splits of K.  For narrow matrices (a gate per head): their few blocks would walk a long K alone."""
+    M, K = x.shape
+    N = weight.shape[0]
+    if gemm_sm100_ok(x, weight):
+        want = min(MAX_RESIDUAL_SPLITS, max(1, sm_count(weight.device) // -(-N // 128)), max(1, -(-K // 64) // 2))
+        s = gemm_splits(K, want)
+        if s > 1:
+            buf = ws.flat(name + "_partials", s * M * N, torch.float32, reserve=MAX_RESIDUAL_SPLITS * min(ws.max_rows, 64) * N)
+            buf = buf[: s * M * N].view(s, M, N)
+            gemm_sm100(x, weight, None, buf, splits=s)
+            return buf
+    out = ws.buf(name, M, N, torch.float32)
+    linear(x, weight, None, out)
     return out
 
 

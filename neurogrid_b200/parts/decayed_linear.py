@@ -141,8 +141,7 @@ class MLSTM(_DecayedLinear):
         state, nm = cache
         p = ctx.ws.buf("dl_in", n, self.w_in.shape[0], self.dtype)
         ops.linear(x, self.w_in, None, p)
-        gates = ctx.ws.buf("dl_gates", n, 2 * s.n_heads, torch.float32)
-        ops.linear(x, self.w_gates, None, gates)
+        gates = ops.linear_f32(x, self.w_gates, ctx.ws, f"dl_gates_{s.n_heads}")
         raw = ctx.ws.buf("dl_raw", n, s.n_heads * s.value_dim, torch.float32)
         ops.mlstm(p, gates, self.b_gates, s.gate_cap, self.norm, state.state, nm.state, raw, out, ctx.cu_q, ctx.ctx_before,
                   ctx.slots, ctx.row_entry, ctx.n_entries, s.n_heads, s.key_dim, s.value_dim, s.eps, out_scale,

@@ -529,6 +529,7 @@ def lightning(x, decay, norm_w, state, o_raw, out, cu_q, ctx_before, slots, row_
 def mlstm(x, gates, gate_bias, cap, norm_w, state, nm_state, o_raw, out, cu_q, ctx_before, slots, row_entry, n_entries,
           n_heads, key_dim, value_dim, eps, out_scale=1.0, scratch=None, max_q=0):
     H, dk, dv = n_heads, key_dim, value_dim
+    gates = gates.sum(0) if gates.dim() == 3 else gates
     pre = cap * torch.tanh((gates.to(D) + gate_bias.to(D)) / cap)
     log_i, log_f = pre[:, :H], torch.nn.functional.logsigmoid(pre[:, H:])
     z = lambda *s: torch.zeros(*s, dtype=D, device=x.device)

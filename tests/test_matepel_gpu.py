@@ -264,7 +264,8 @@ def _mlstm_inputs(dtype, T, H, dk, dv, seed=0):
 class _Recurrence:
     """One of the two recurrences on its own: inputs, the kernels, the plain statement, states."""
 
-    def __init__(self, kind, dtype, T, H, dk, dv, seed=0, cap=6.0):
+    def __init__(self, kind, dtype, T, H, dk, dv, seed=0, cap=6.0, parts=1):
+        self.parts = parts
         self.kind, self.dtype, self.H, self.dk, self.dv, self.cap = kind, dtype, H, dk, dv, cap
         if kind == "lightning":
             self.x, self.decay, self.nw = _lightning_inputs(dtype, T, H, dk, dv, seed)      # (a decay per head)
@@ -291,7 +292,11 @@ class _Recurrence:
         if self.kind == "lightning":
             ops().lightning(x, ops().decay_powers(self.decay, DEV), self.nw, states[0], raw, *tail, **kw)
         else:
-            ops().mlstm(x, self.gates[rows].contiguous(), self.bias, self.cap, self.nw, states[0], states[1], raw, *tail, **kw)
+            gates = self.gates[rows].contiguous()
+            if self.parts > 1:                             # the same numbers as a stack of partial sums
+                cut = torch.randn(self.parts - 1, *gates.shape, generator=torch.Generator().manual_seed(1)).to(DEV)
+                gates = torch.cat([cut, (gates - cut.sum(0))[None]]).contiguous()
+            ops().mlstm(x, gates, self.bias, self.cap, self.nw, states[0], states[1], raw, *tail, **kw)
 
     def plain(self, rows, states=None, scale=1.0):
         """(output, states) of consecutive rows of one request, float64."""
@@ -347,7 +352,7 @@ def test_recurrence_whole_cut_and_token_by_token(kind, dtype, H, dk, dv):
 def test_recurrence_batch_of_unequal_entries(kind, dtype, chunked):
     H, dk, dv = 3, 32, 48
     lens, before, slots = [1, 37, 2, 200, 64], [5, 0, 40, 12, 0], [3, 0, 2, 1, 4]
-    r = _Recurrence(kind, dtype, sum(lens), H, dk, dv, seed=4)
+    r = _Recurrence(kind, dtype, sum(lens), H, dk, dv, seed=4, parts=3)
     states = r.states(5, seed=8)
     first = [s.clone() for s in states]
     ctx = make_ctx(lens, before, slots, dtype=dtype)
