@@ -125,7 +125,7 @@ def test_specs_refuse_what_no_kernel_does():
     dict(base=50.0, dims=4, scaling=dict(factor=2.0, original=300, fast=20.0, slow=2.0)),
     dict(base=10.0, dims=4, scaling=dict(factor=4.0, original=4, fast=6.0, slow=5.0)),            # both edges at the start
     dict(base=100.0, dims=32, scaling=dict(factor=3.0, original=100000, fast=2.0, slow=1.0)),     # nothing is divided
-    dict(base=1e6, dims=64, scaling=dict(factor=1.0, original=2048, fast=32.0, slow=1.0)),
+    dict(base=1e6, dims=64, scaling=dict(factor=1.0, original=1536, fast=40.0, slow=2.0)),
 ])
 def test_rescaled_frequencies(rot):
     sc = rot["scaling"]
