@@ -18,6 +18,7 @@ from .rofulorn import RofulornConfig
 from .fuzelorn import FuzelornConfig
 from .dodilix import DodilixConfig
 from .matepel import MatepelConfig
+from .pepulix import PepulixConfig
 
 _ARCHITECTURES: Dict[str, Any] = {}
 _MODEL_TYPES: Dict[str, str] = {}
@@ -68,3 +69,4 @@ register_architecture("Rofulorn", RofulornConfig)
 register_architecture("Fuzelorn", FuzelornConfig)
 register_architecture("Dodilix", DodilixConfig)
 register_architecture("Matepel", MatepelConfig)
+register_architecture("Pepulix", PepulixConfig)

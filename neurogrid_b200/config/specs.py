@@ -149,6 +149,12 @@ class MappedAttentionSpec:
     one more projection of the mixer's input (rows ``g``) before the output projection.  ``unit_sink``: the softmax's
     denominator holds one more 1, a sink whose score is 0 for every head (nothing is learned).  ``shared_kv``: there is
     no v projection, the values are the keys as projected (with their bias, before norm and ``position``).
+    ``weights`` "sigmoid" (one map): no softmax; a visible key's weight is sigmoid(s + b_h) with a stored number b_h per
+    head (``score_bias``), not normalised over the keys.  ``value_norm``: every value head over its root mean square
+    (``eps``, no weight).  ``value_mix``: "source": the layer's values (normed, if ``value_norm``) are kept for the layers of the
+    same step with "mix", whose values become (1 - lambda) v + lambda v_source with a stored lambda (``vmix``); the mixed
+    values are what is cached ("source" stores a lambda too, unused).  ``head_gate``: head h's output is multiplied by
+    sigmoid(W_g x)_h, one number per head.  ``o_bias`` False: q, k and v have biases and the output projection has none.
     """
     hidden: int
     n_heads: int
@@ -176,9 +182,16 @@ class MappedAttentionSpec:
     out_gate: bool = False
     unit_sink: bool = False
     shared_kv: bool = False
+    weights: str = "softmax"
+    score_bias: bool = False
+    value_norm: bool = False
+    value_mix: Optional[str] = None
+    head_gate: bool = False
+    o_bias: bool = True
     names: Mapping[str, str] = field(default_factory=lambda: _names(
         q="q", k="k", v="v", o="o", q_bias="q.b", k_bias="k.b", v_bias="v.b", o_bias="o.b", q_norm="q.norm",
-        k_norm="k.norm", lq1="lq1", lk1="lk1", lq2="lq2", lk2="lk2", sink="sink", out_gate="g"))
+        k_norm="k.norm", lq1="lq1", lk1="lk1", lq2="lq2", lk2="lk2", sink="sink", out_gate="g", head_gate="g",
+        score_bias="pb", value_mix="vmix"))
     kind: str = "mapped_attention"
 
     def __post_init__(self):
@@ -204,6 +217,16 @@ class MappedAttentionSpec:
             raise ValueError("values that are the keys have the keys' size and one map")
         if self.qk_norm and not self.norm_weight and getattr(self.position, "yarn", None) is not None:
             raise ValueError("a norm without weights goes with a rotation that keeps lengths")
+        if self.weights not in ("softmax", "sigmoid") or (self.score_bias and self.weights != "sigmoid"):
+            raise ValueError("attention weights are softmax or sigmoid, and a bias per head goes with sigmoid")
+        if self.weights == "sigmoid" and (self.n_maps != 1 or self.sink or self.unit_sink):
+            raise ValueError("sigmoid weights have one map per head and no sink")
+        if self.value_mix not in (None, "source", "mix"):
+            raise ValueError("value_mix is None, source or mix")
+        if (self.value_norm or self.value_mix) and self.shared_kv:
+            raise ValueError("values that are the keys are neither normed nor mixed")
+        if self.head_gate and self.out_gate:
+            raise ValueError("an output gate is per head or per coordinate")
 
 
 @dataclass(frozen=True)
@@ -225,7 +248,8 @@ class ShortConvSpec:
 class SwiGLUSpec:
     """down( act(gate(x)) * up(x) ), no biases; ``activation`` "silu" or "gelu_tanh" (the tanh form of gelu), or
     "clamped_glu": g sigmoid(``glu_alpha`` g) (u + 1) with g = min(gate(x), limit), u = clamp(up(x), -limit, limit).
-    A tensor's name is its role's name plus ``weight_suffix``."""
+    A tensor's name is its role's name plus ``weight_suffix``.  ``bias``: all three projections have one, stored under the
+    projection's name plus ``bias_suffix``."""
     hidden: int
     intermediate: int
     names: Mapping[str, str] = field(default_factory=lambda: _names(
@@ -234,6 +258,8 @@ class SwiGLUSpec:
     weight_suffix: str = ".weight"
     limit: float = 0.0
     glu_alpha: float = 1.702
+    bias: bool = False
+    bias_suffix: str = ".b"
     kind: str = "swiglu"
 
     def __post_init__(self):
@@ -288,7 +314,7 @@ class LatentAttentionSpec:
     ``rope_dim`` r > 0: q has r more coordinates per head (laid out [key_dim | r]) and W_dkv r more rows, one key
     part shared by all heads and not normed; both are rotated by ``position`` (over all r coordinates) and the score
     is the sum of the two dot products.  The latent and the rotated key part are cached.  ``gate`` "element": the
-    gate has a row per coordinate of the concatenated heads instead of one per head.
+    gate has a row per coordinate of the concatenated heads instead of one per head; "none": there is no gate.
     """
     hidden: int
     n_heads: int
@@ -309,12 +335,12 @@ class LatentAttentionSpec:
     def __post_init__(self):
         if self.window is not None and self.window < 1:
             raise ValueError("attention window must be >= 1")
-        if not (1 <= self.kv_rank <= 512):
-            raise ValueError(f"latent attention: kv_rank must be in [1, 512], got {self.kv_rank}")
+        if self.kv_rank < 1 or self.kv_rank + self.rope_dim > 768:
+            raise ValueError(f"latent attention: kv_rank and the rotated key part must be in 1..768 together, got {self.kv_rank} + {self.rope_dim}")
         if self.rope_dim < 0 or self.rope_dim % 2 or (self.rope_dim > 0) != (self.position is not None):
             raise ValueError("latent attention: a rotated key part has an even size and a position encoding")
-        if self.gate not in ("head", "element"):
-            raise ValueError("latent attention: the gate is per head or per element")
+        if self.gate not in ("head", "element", "none"):
+            raise ValueError("latent attention: the gate is per head, per element or none")
 
 
 @dataclass(frozen=True)
@@ -332,7 +358,9 @@ class MoESpec:
     ``shared_gate``: the shared expert's output is multiplied by sigmoid(w . x), one number per token.
     ``scoring`` "softmax_all": scores s = softmax(logits) over ALL experts, no bias, and then as for sigmoid scores
     (correction, groups, s over the chosen sum).  ``group_score`` "top2" (the sum of a group's two largest choice
-    scores) or "max".  ``route_scale`` multiplies the routing weights."""
+    scores) or "max".  ``route_scale`` multiplies the routing weights.
+    ``identity`` n > 0 (sigmoid or softmax_all scoring): the router has n more outputs behind the experts'; they are scored
+    and chosen with them, and stand for experts without tensors whose output is the input itself."""
     hidden: int
     n_experts: int
     top_k: int
@@ -349,14 +377,18 @@ class MoESpec:
     shared_gate: bool = False
     group_score: str = "top2"
     route_scale: float = 1.0
+    identity: int = 0
     names: Mapping[str, str] = field(default_factory=lambda: _names(
         expert="e{}", gate="gate", up="up", down="down", router="router", router_bias="router.b", shared="shared",
         correction="correction", shared_gate="shared.sg"))
     kind: str = "moe"
 
     def __post_init__(self):
-        if not (1 <= self.top_k <= self.n_experts):
-            raise ValueError(f"moe: top_k {self.top_k} must be in 1..{self.n_experts}")
+        n_routed = self.n_experts + self.identity
+        if self.identity < 0 or (self.identity and self.scoring == "softmax"):
+            raise ValueError("moe: identity experts go with sigmoid or softmax_all scoring")
+        if not (1 <= self.top_k <= n_routed):
+            raise ValueError(f"moe: top_k {self.top_k} must be in 1..{n_routed}")
         if self.top_k > 32:
             raise ValueError("moe: top_k above 32 is not supported")
         if self.scoring not in ("softmax", "sigmoid", "softmax_all") or self.activation not in ("swiglu", "clamped_glu"):
@@ -365,9 +397,9 @@ class MoESpec:
             raise ValueError("moe: a group's score is top2 or max")
         if self.scoring == "softmax" and self.route_scale != 1.0:
             raise ValueError("moe: a scale of the routing weights goes with sigmoid or softmax_all scoring")
-        if self.n_groups < 1 or self.n_experts % self.n_groups or not (1 <= self.keep_groups <= self.n_groups):
-            raise ValueError(f"moe: {self.n_experts} experts do not form {self.n_groups} equal groups of which {self.keep_groups} are kept")
-        if self.top_k > self.keep_groups * (self.n_experts // self.n_groups):
+        if self.n_groups < 1 or n_routed % self.n_groups or not (1 <= self.keep_groups <= self.n_groups):
+            raise ValueError(f"moe: {n_routed} experts do not form {self.n_groups} equal groups of which {self.keep_groups} are kept")
+        if self.top_k > self.keep_groups * (n_routed // self.n_groups):
             raise ValueError("moe: the kept groups hold fewer experts than top_k")
         if self.scoring == "softmax" and (self.correction or self.n_groups > 1):
             raise ValueError("moe: a correction and groups go with sigmoid scoring")

@@ -13,9 +13,10 @@
 #include "ng_common.cuh"
 
 #define AG_WARPS 4
-#define AG_MAX_J 16     // head_dim <= 512
+#define AG_MAX_J 24     // head_dim <= 768
 
-template <typename T>
+// MJ: columns a lane holds (head_dim <= 32 * MJ)
+template <typename T, int MJ>
 __global__ void __launch_bounds__(AG_WARPS * 32)
 attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages, const T* __restrict__ v_pages,
                          const int* __restrict__ table, int table_stride, const int* __restrict__ positions,
@@ -38,9 +39,9 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
     const int lo = window > 0 ? max(0, pos - window + 1) : 0;
     const float slope = slopes ? slopes[head] : 0.f;          // score bias: -slope * (query position - key position)
     const T* qr = q + ((size_t)row * nH + head) * hd;
-    float qv[AG_MAX_J], acc[AG_MAX_J];
+    float qv[MJ], acc[MJ];
 #pragma unroll
-    for (int j = 0; j < AG_MAX_J; ++j) {
+    for (int j = 0; j < MJ; ++j) {
         const int d = lane + 32 * j;
         qv[j] = d < hd ? ng_ld(qr + d) * scale : 0.f;
         acc[j] = 0.f;
@@ -53,7 +54,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
         const size_t base = (((size_t)page * nKV + kvh) * page_size + (kp % page_size)) * hd;
         float dot = 0.f;
 #pragma unroll
-        for (int j = 0; j < AG_MAX_J; ++j) {
+        for (int j = 0; j < MJ; ++j) {
             const int d = lane + 32 * j;
             if (d < hd) dot = fmaf(qv[j], ng_ld(k_pages + base + d), dot);
         }
@@ -63,7 +64,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
         const float p = expf(s - m_new);
         l = l * corr + p;
 #pragma unroll
-        for (int j = 0; j < AG_MAX_J; ++j) {
+        for (int j = 0; j < MJ; ++j) {
             const int d = lane + 32 * j;
             if (d < hd) acc[j] = acc[j] * corr + p * ng_ld(v_pages + base + d);
         }
@@ -71,7 +72,7 @@ attention_generic_kernel(const T* __restrict__ q, const T* __restrict__ k_pages,
     }
     const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
-    for (int j = 0; j < AG_MAX_J; ++j) {
+    for (int j = 0; j < MJ; ++j) {
         const int d = lane + 32 * j;
         if (d < hd) ng_st(o + d, acc[j] * inv);
     }
@@ -84,13 +85,16 @@ NG_EXPORT int ng_attention_generic(const void* q, const void* k_pages, const voi
     if (n_rows <= 0) return NG_OK;
     if (hd <= 0 || hd > 32 * AG_MAX_J || nH <= 0 || nKV <= 0 || nH % nKV || page_size <= 0) return NG_BAD_SIZE;
     dim3 grid(n_rows, (nH + AG_WARPS - 1) / AG_WARPS);
-    if (act_bf16)
-        NG_LAUNCH((attention_generic_kernel<__nv_bfloat16>), grid, AG_WARPS * 32, 0, stream, 
-            (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pages, (const __nv_bfloat16*)v_pages, table,
-            table_stride, positions, row_entry, (__nv_bfloat16*)out, nH, nKV, hd, page_size, num_pages, window, scale, slopes);
-    else
-        NG_LAUNCH((attention_generic_kernel<float>), grid, AG_WARPS * 32, 0, stream, 
-            (const float*)q, (const float*)k_pages, (const float*)v_pages, table, table_stride, positions,
-            row_entry, (float*)out, nH, nKV, hd, page_size, num_pages, window, scale, slopes);
+#define AG_LAUNCH(TT, MJ)                                                                                              \
+    NG_LAUNCH((attention_generic_kernel<TT, MJ>), grid, AG_WARPS * 32, 0, stream, (const TT*)q, (const TT*)k_pages,    \
+              (const TT*)v_pages, table, table_stride, positions, row_entry, (TT*)out, nH, nKV, hd, page_size, num_pages, \
+              window, scale, slopes)
+    if (act_bf16) {
+        if (hd <= 512) AG_LAUNCH(__nv_bfloat16, 16);
+        else AG_LAUNCH(__nv_bfloat16, 24);
+    } else {
+        if (hd <= 512) AG_LAUNCH(float, 16);
+        else AG_LAUNCH(float, 24);
+    }
     return ng_launch_status();
 }

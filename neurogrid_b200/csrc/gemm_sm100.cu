@@ -31,7 +31,7 @@
 // ------------------------------------------------------------------------------------- kernel
 struct GemmParams {
     void* out;                 // bf16 [M, ldc] | float [splits][M, ldc]
-    const bf16* bias;          // [N] or null (EPI_BF16 only)
+    const bf16* bias;          // [N] or null (EPI_BF16; EPI_SWIGLU: per row of W, gate and up)
     int* status;
     int M, N, K;               // N = rows of W that produce outputs (for SwiGLU: the intermediate size I)
     int ldc;
@@ -199,6 +199,8 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
         const int tl = warp * 32 + lane;                        // this thread's TMEM lane
         const int peer = up_half ? tl - 64 : tl + 64;
         const int j0 = up_half ? 8 : 0;                         // tokens of the chunk this thread finishes
+        float bg = 0.f, bu = 0.f;                               // biases of the gate and the up column
+        if (p.bias && col < p.rows && n < p.N) { bg = __bfloat162float(p.bias[n]); bu = __bfloat162float(p.bias[p.up_row_offset + n]); }
 #pragma unroll 1
         for (int c = 0; c < TN; c += 16) {
             float v[16];
@@ -213,8 +215,8 @@ gemm_sm100_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
                     if (m < p.M) {
                         const float mine = up_half ? v[8 + j] : v[j], theirs = xch[peer][j0 + j];
                         // the unfused path rounds both products to bf16 before the gate: keep that rounding
-                        const float g = __bfloat162float(__float2bfloat16_rn(up_half ? theirs : mine));
-                        const float u = __bfloat162float(__float2bfloat16_rn(up_half ? mine : theirs));
+                        const float g = __bfloat162float(__float2bfloat16_rn((up_half ? theirs : mine) + bg));
+                        const float u = __bfloat162float(__float2bfloat16_rn((up_half ? mine : theirs) + bu));
                         float y;
                         if (p.gate_kind == 2) {
                             const float gc = fminf(g, p.gate_limit);
@@ -312,7 +314,8 @@ static int dispatch_tn(int tn, const CUtensorMap& mw, const CUtensorMap& mx, con
 // x [M,K] bf16, w [n_w_rows,K] bf16 (both row-major, 16-byte aligned, K % 8 == 0).
 //   epi 0: out bf16 [M, ldc] = x w^T (+ bias)              N = n_w_rows, splits must be 1
 //   epi 1: out float [splits][M, ldc] = partial x w^T      N = n_w_rows
-//   epi 2: out bf16 [M, ldc] = silu(x wg^T) * (x wu^T)     wg = w rows [0, N), wu = w rows [up_row_offset, +N)
+//   epi 2: out bf16 [M, ldc] = silu(x wg^T) * (x wu^T)     wg = w rows [0, N), wu = w rows [up_row_offset, +N); bias
+//          [n_w_rows] or null is added to both products before they are rounded
 //   epi 3: out float [M, ldc] += x w^T (atomic adds; any splits)
 //   epi 4: as epi 2 with gelu_tanh(z) = 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3))) for silu
 //   epi 5: as epi 0, then relu(.)^2 of the rounded result

@@ -7,7 +7,8 @@
 //   2. with `delta` (the output y of the sublayer before: [n, H] of the activation type, or float32 partial sums that
 //      are added in ascending order) all streams are replaced at once from the old ones,
 //          x_t <- sum_s mix[s, t] x_s + out_w[t] * y            (mix is indexed [from, to]);
-//      `bias` [H] (float32, optional) belongs to y: it is added to delta's value;
+//      `bias` [H] (float32, optional) belongs to y: it is added to delta's value, and so is (optional) id_w[row] * id_x[row],
+//      a multiple of what that sublayer read (id_x [n, H] of the activation type, id_w rows id_ld apart);
 //   3. with `in_w`: u = sum_t in_w[t] x_t is what the next sublayer reads, and `out` receives
 //      u / sqrt(mean(u^2) + eps) * norm_w in the activation type (one rounding);
 //   4. with `sum_out`: the sum of the streams (float32 [n, H]), which is what the model's last norm reads.
@@ -23,7 +24,8 @@ __global__ void __launch_bounds__(512)
 hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __restrict__ delta, int n_partials,
                size_t partial_stride, const float* __restrict__ mix, const float* __restrict__ out_w,
                const float* __restrict__ in_w, const float* __restrict__ norm_w, TO* __restrict__ out,
-               float* __restrict__ sum_out, const float* __restrict__ bias, int S_rt, int H, float eps) {
+               float* __restrict__ sum_out, const float* __restrict__ bias, const TO* id_x, const float* id_w, int id_ld, int S_rt,
+               int H, float eps) {
     extern __shared__ float u_s[];                     // [H]: what the next sublayer reads, before its norm
     __shared__ float red[32];
     __shared__ float mix_s[HC_MAX_STREAMS * HC_MAX_STREAMS], ow_s[HC_MAX_STREAMS], iw_s[HC_MAX_STREAMS];
@@ -39,7 +41,9 @@ hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __
     ng_pdl_wait();
     delta = ng_after_wait(delta);
     x0 = ng_after_wait(x0);
+    id_x = ng_after_wait(id_x);
     const size_t row = blockIdx.x;
+    const float idw = id_x ? *ng_after_wait(id_w + row * id_ld) : 0.f;
     float* xr = X + row * (size_t)S * H;
     float ss = 0.f;
     for (int j = threadIdx.x * VEC; j < H; j += blockDim.x * VEC) {
@@ -74,6 +78,7 @@ hc_step_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __
                 y[v] = 0.f;
                 for (int p = 0; p < n_partials; ++p) y[v] += ng_ld(delta + p * partial_stride + row * H + j + v);   // ascending p
                 if (bias) y[v] += bias[j + v];
+                if (id_x) y[v] = fmaf(idw, ng_ld(id_x + row * H + j + v), y[v]);
             }
             float nx[SM][VEC];
 #pragma unroll
@@ -152,7 +157,7 @@ __global__ void __launch_bounds__(512)
 hc_step_row_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD* __restrict__ delta, int n_partials,
                    size_t partial_stride, const float* __restrict__ mix, const float* __restrict__ out_w,
                    const float* __restrict__ in_w, const float* __restrict__ norm_w, TO* __restrict__ out,
-                   float* __restrict__ sum_out, const float* __restrict__ bias, int H, float eps) {
+                   float* __restrict__ sum_out, const float* __restrict__ bias, const TO* id_x, const float* id_w, int id_ld, int H, float eps) {
     __shared__ float red[32];
     __shared__ float mix_s[S * S], ow_s[S], iw_s[S];
     ng_pdl_trigger();
@@ -170,7 +175,9 @@ hc_step_row_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD
     ng_pdl_wait();
     delta = ng_after_wait(delta);
     x0 = ng_after_wait(x0);
+    id_x = ng_after_wait(id_x);
     const size_t row = blockIdx.x;
+    const float idw = id_x ? *ng_after_wait(id_w + row * id_ld) : 0.f;
     float* xr = X + row * (size_t)S * H + j;
     float4 xs[S], u = zero;
     if (live) {
@@ -190,6 +197,10 @@ hc_step_row_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD
                 a.x += t.x; a.y += t.y; a.z += t.z; a.w += t.w;
             }
             y.x += a.x; y.y += a.y; y.z += a.z; y.w += a.w;
+            if (id_x) {
+                const float4 t = hc_ld4(id_x + row * H + j);
+                y.x = fmaf(idw, t.x, y.x); y.y = fmaf(idw, t.y, y.y); y.z = fmaf(idw, t.z, y.z); y.w = fmaf(idw, t.w, y.w);
+            }
             float4 nx[S];
 #pragma unroll
             for (int t = 0; t < S; ++t) {
@@ -231,8 +242,8 @@ hc_step_row_kernel(float* __restrict__ X, const float* __restrict__ x0, const TD
 
 template <typename TD, typename TO, int S_CT, int VEC>
 static int hc_launch(float* X, const float* x0, const void* delta, int n_partials, size_t ps, const float* mix,
-                     const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
-                     int H, float eps, cudaStream_t stream) {
+                     const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, const void* id_x,
+                     const float* id_w, int id_ld, int n_rows, int S, int H, float eps, cudaStream_t stream) {
     static bool configured = false;
     if (!configured) {
         if (cudaFuncSetAttribute(hc_step_kernel<TD, TO, S_CT, VEC>, cudaFuncAttributeMaxDynamicSharedMemorySize, 160 * 1024) !=
@@ -246,49 +257,50 @@ static int hc_launch(float* X, const float* x0, const void* delta, int n_partial
     int threads = n_rows <= 64 ? 512 : 256;
     while (threads > 64 && threads / 2 >= per) threads /= 2;
     NG_LAUNCH((hc_step_kernel<TD, TO, S_CT, VEC>), n_rows, threads, smem, stream, X, x0, (const TD*)delta, n_partials, ps, mix,
-              out_w, in_w, norm_w, (TO*)out, sum_out, bias, S, H, eps);
+              out_w, in_w, norm_w, (TO*)out, sum_out, bias, (const TO*)id_x, id_w, id_ld, S, H, eps);
     return ng_launch_status();
 }
 
 template <typename TD, typename TO>
 static int hc_by_streams(float* X, const float* x0, const void* delta, int n_partials, size_t ps, const float* mix,
-                         const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S,
-                         int H, float eps, cudaStream_t stream) {
+                         const float* out_w, const float* in_w, const float* norm_w, void* out, float* sum_out, const float* bias, const void* id_x,
+                         const float* id_w, int id_ld, int n_rows, int S, int H, float eps, cudaStream_t stream) {
     const bool vec = H % 4 == 0 && ((uintptr_t)X & 15) == 0;
     // rows that a block holds at once: four columns a thread, at most 512 threads
     const bool row_at_once = vec && H <= 2048 && ps % 4 == 0 && ((uintptr_t)delta % (4 * sizeof(TD))) == 0 &&
-                             ((uintptr_t)out % (4 * sizeof(TO))) == 0 &&
+                             ((uintptr_t)out % (4 * sizeof(TO))) == 0 && ((uintptr_t)id_x % (4 * sizeof(TO))) == 0 &&
                              (((uintptr_t)x0 | (uintptr_t)sum_out | (uintptr_t)norm_w | (uintptr_t)bias) & 15) == 0;
 #define HC_CASE(SS)                                                                                                    \
     case SS:                                                                                                           \
         if (row_at_once) {                                                                                             \
             NG_LAUNCH((hc_step_row_kernel<TD, TO, SS>), n_rows, (H / 4 + 31) / 32 * 32, 0, stream, X, x0, (const TD*)delta, \
-                      n_partials, ps, mix, out_w, in_w, norm_w, (TO*)out, sum_out, bias, H, eps);                      \
+                      n_partials, ps, mix, out_w, in_w, norm_w, (TO*)out, sum_out, bias, (const TO*)id_x, id_w, id_ld, H, eps); \
             return ng_launch_status();                                                                                 \
         }                                                                                                              \
-        return vec ? hc_launch<TD, TO, SS, 4>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream) \
-                   : hc_launch<TD, TO, SS, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
+        return vec ? hc_launch<TD, TO, SS, 4>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream) \
+                   : hc_launch<TD, TO, SS, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream);
     switch (S) {
         HC_CASE(1) HC_CASE(2) HC_CASE(3) HC_CASE(4) HC_CASE(5) HC_CASE(6) HC_CASE(7) HC_CASE(8)
         default:
-            return hc_launch<TD, TO, 0, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
+            return hc_launch<TD, TO, 0, 1>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream);
     }
 }
 
 // delta: null, one [n, H] tensor of the activation type, or (delta_f32) n_partials float32 tensors [n, H] that lie
-// partial_stride elements apart.  x0, in_w (with norm_w and out), sum_out and bias are optional; mix and out_w go with delta.
+// partial_stride elements apart.  x0, in_w (with norm_w and out), sum_out, bias and id_x (with id_w; another buffer than out)
+// are optional; mix and out_w go with delta.
 NG_EXPORT int ng_hc_step(float* X, const float* x0, const void* delta, int delta_f32, int n_partials,
                          long long partial_stride, const float* mix, const float* out_w, const float* in_w,
-                         const float* norm_w, void* out, float* sum_out, const float* bias, int n_rows, int S, int H, float eps,
-                         int act_bf16, cudaStream_t stream) {
+                         const float* norm_w, void* out, float* sum_out, const float* bias, const void* id_x,
+                         const float* id_w, int id_ld, int n_rows, int S, int H, float eps, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (S < 1 || S > HC_MAX_STREAMS || H <= 0 || n_partials < 1 || (delta && (!mix || !out_w)) || (in_w && (!norm_w || !out)) ||
-        (size_t)H * sizeof(float) > 160 * 1024)
+        (size_t)H * sizeof(float) > 160 * 1024 || (id_x && (!id_w || !delta || id_ld < 1 || id_x == out)))
         return NG_BAD_SIZE;
     const size_t ps = (size_t)partial_stride;
     if (act_bf16 && delta_f32)
-        return hc_by_streams<float, __nv_bfloat16>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
+        return hc_by_streams<float, __nv_bfloat16>(X, x0, delta, n_partials, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream);
     if (act_bf16)
-        return hc_by_streams<__nv_bfloat16, __nv_bfloat16>(X, x0, delta, 1, 0, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
-    return hc_by_streams<float, float>(X, x0, delta, delta_f32 ? n_partials : 1, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, n_rows, S, H, eps, stream);
+        return hc_by_streams<__nv_bfloat16, __nv_bfloat16>(X, x0, delta, 1, 0, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream);
+    return hc_by_streams<float, float>(X, x0, delta, delta_f32 ? n_partials : 1, ps, mix, out_w, in_w, norm_w, out, sum_out, bias, id_x, id_w, id_ld, n_rows, S, H, eps, stream);
 }

@@ -6,7 +6,8 @@
 //                                                             [pages, 1, page_size, rp], columns rkv+rot..rp zero
 //   key part (rot columns, not normed), rotated by the row's position: pair i is (2i, 2i+1) or, with half
 //   pairing, (i, i + rot/2), its angle position * inv_freq[i]  -> columns rkv..rkv+rot of the same place
-//   gate = sigmoid(gate logits)                             -> gate_out [n_rows, nH]    (float32; nH: gate columns)
+//   (cosines and sines times rot_mag)
+//   gate = sigmoid(gate logits)                             -> gate_out [n_rows, nH]    (float32; nH: gate columns, 0: no gate)
 // rkv = 0 (no pages): a layer that reads another layer's latents.
 // Both norms, the angles and the gate are float32; only what a matrix product or the cache reads is rounded.
 //
@@ -25,7 +26,8 @@ latent_prep_kernel(const T* __restrict__ x, const float* __restrict__ wq, const 
                    T* __restrict__ cq_out, T* __restrict__ pages, float* __restrict__ gate_out,
                    const int* __restrict__ table, int table_stride, const int* __restrict__ positions,
                    const int* __restrict__ row_entry, int rq, int rkv, int rp, int nH, int page_size, int num_pages,
-                   float eps, int* __restrict__ status, int rot, const float* __restrict__ inv_freq, int half_pairing) {
+                   float eps, int* __restrict__ status, int rot, const float* __restrict__ inv_freq, int half_pairing,
+                   float rot_mag) {
     __shared__ float red[32];
     ng_pdl_trigger();
     ng_pdl_wait();
@@ -62,6 +64,7 @@ latent_prep_kernel(const T* __restrict__ x, const float* __restrict__ wq, const 
                 const int c1 = half_pairing ? i : 2 * i, c2 = half_pairing ? i + rot / 2 : 2 * i + 1;
                 float sn, cs;
                 sincosf((float)pos * inv_freq[i], &sn, &cs);
+                sn *= rot_mag; cs *= rot_mag;
                 const float a = ng_ld(kr + c1), b = ng_ld(kr + c2);
                 ng_st(dst + rkv + c1, a * cs - b * sn);
                 ng_st(dst + rkv + c2, b * cs + a * sn);
@@ -74,7 +77,8 @@ latent_prep_kernel(const T* __restrict__ x, const float* __restrict__ wq, const 
 
 template <typename T>
 __global__ void latent_rope_q_kernel(T* __restrict__ q, const int* __restrict__ positions, const int* __restrict__ row_entry,
-                                     const float* __restrict__ inv_freq, int nH, int rp, int off, int rot, int half_pairing) {
+                                     const float* __restrict__ inv_freq, int nH, int rp, int off, int rot, int half_pairing,
+                                     float rot_mag) {
     ng_pdl_trigger();
     ng_pdl_wait();
     const int row = blockIdx.x;
@@ -88,6 +92,7 @@ __global__ void latent_rope_q_kernel(T* __restrict__ q, const int* __restrict__ 
         T* p = qr + (size_t)h * rp + off;
         float sn, cs;
         sincosf(pos * inv_freq[i], &sn, &cs);
+        sn *= rot_mag; cs *= rot_mag;
         const float a = ng_ld(p + c1), b = ng_ld(p + c2);
         ng_st(p + c1, a * cs - b * sn);
         ng_st(p + c2, b * cs + a * sn);
@@ -382,32 +387,32 @@ NG_EXPORT int ng_latent_prep(const void* x, const float* wq, const float* wkv, v
                              float* gate_out, const int* table, int table_stride, const int* positions,
                              const int* row_entry, int n_rows, int rq, int rkv, int rp, int nH, int page_size,
                              int num_pages, float eps, int* status, int rot, const float* inv_freq, int half_pairing,
-                             int act_bf16, cudaStream_t stream) {
+                             float rot_mag, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
-    if (rq <= 0 || rkv < 0 || rot < 0 || (rot & 1) || (rot && !inv_freq) || (rkv == 0 && rot) || rp < rkv + rot || nH <= 0 ||
-        page_size <= 0 || (rkv > 0 && !pages))
+    if (rq <= 0 || rkv < 0 || rot < 0 || (rot & 1) || (rot && !inv_freq) || (rkv == 0 && rot) || rp < rkv + rot || nH < 0 ||
+        (nH > 0 && !gate_out) || page_size <= 0 || (rkv > 0 && !pages))
         return NG_BAD_SIZE;
     if (act_bf16)
         NG_LAUNCH((latent_prep_kernel<__nv_bfloat16>), n_rows, 128, 0, stream, (const __nv_bfloat16*)x, wq, wkv,
                   (__nv_bfloat16*)cq_out, (__nv_bfloat16*)pages, gate_out, table, table_stride, positions, row_entry,
-                  rq, rkv, rp, nH, page_size, num_pages, eps, status, rot, inv_freq, half_pairing);
+                  rq, rkv, rp, nH, page_size, num_pages, eps, status, rot, inv_freq, half_pairing, rot_mag);
     else
         NG_LAUNCH((latent_prep_kernel<float>), n_rows, 128, 0, stream, (const float*)x, wq, wkv, (float*)cq_out,
                   (float*)pages, gate_out, table, table_stride, positions, row_entry, rq, rkv, rp, nH, page_size,
-                  num_pages, eps, status, rot, inv_freq, half_pairing);
+                  num_pages, eps, status, rot, inv_freq, half_pairing, rot_mag);
     return ng_launch_status();
 }
 
 NG_EXPORT int ng_latent_rope_q(void* q, const int* positions, const int* row_entry, const float* inv_freq, int n_rows,
-                               int nH, int rp, int off, int rot, int half_pairing, int act_bf16, cudaStream_t stream) {
+                               int nH, int rp, int off, int rot, int half_pairing, float rot_mag, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0 || rot == 0) return NG_OK;
     if (nH <= 0 || rp <= 0 || off < 0 || rot < 0 || (rot & 1) || off + rot > rp || !inv_freq) return NG_BAD_SIZE;
     if (act_bf16)
         NG_LAUNCH((latent_rope_q_kernel<__nv_bfloat16>), n_rows, 128, 0, stream, (__nv_bfloat16*)q, positions, row_entry,
-                  inv_freq, nH, rp, off, rot, half_pairing);
+                  inv_freq, nH, rp, off, rot, half_pairing, rot_mag);
     else
         NG_LAUNCH((latent_rope_q_kernel<float>), n_rows, 128, 0, stream, (float*)q, positions, row_entry, inv_freq, nH, rp,
-                  off, rot, half_pairing);
+                  off, rot, half_pairing, rot_mag);
     return ng_launch_status();
 }
 

@@ -10,12 +10,16 @@
 //   slopes (per head, optional): slope_h * (pos - j) is taken off s(j) after the cap
 //   sinks (per head, optional): the softmax's denominator also holds exp(sink_h), a term without key or value
 //   head_norm: o <- o * rsqrt(mean(o^2) + eps)  over the head's dv values;   then o <- o * post_scale
+//   sigmoid (one map): no softmax; a visible key's weight is sigmoid(s + score_bias[head]) and o the plain weighted sum
+//   gate (optional, [N, .] of the activation type, rows gate_ld apart): o <- o * sigmoid(gate[row, head])
 //
 // Two kernels.  ``qkv_prep``: per-head RMS norm of q and k (one weight vector shared by heads and maps; or, `whole`,
 // one norm over all of a row's q and one over all of its k, with weights of that length), q times a temperature
 // 1 + coef * ln(floor((pos + 1) / every) + 1), rotation of the first rot_dims coordinates of every map in pairs (2i, 2i+1) or
 // (i, i + rot_dims/2), cosine and sine times `rot_mag`, q to its buffer, k and v into
-// their pages (`v_is_k`: the values are the keys as projected, without norm and rotation).  ``mapped_attention``: a block per (row, query head, run of keys); a warp takes 32 keys of a
+// their pages (`v_is_k`: the values are the keys as projected, without norm and rotation; `v_norm`: every value head over
+// its root mean square; `v_mode` 1: the values, float32, also go to `v_first` [N, nV * dv], 2: they become
+// (1 - v_lambda) v + v_lambda v_first before they are stored).  ``mapped_attention``: a block per (row, query head, run of keys); a warp takes 32 keys of a
 // 128-key tile with a lane per key for the scores of both maps (the key's row read in 16-byte pieces, q from
 // shared memory), keeps an online softmax per map in float32 and adds the weighted values with a lane per pair
 // of value columns; the warps' states are merged in warp order, the runs (few-row steps cut a row's keys into
@@ -36,7 +40,8 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
                 T* __restrict__ k_pages, T* __restrict__ v_pages, const int* __restrict__ table, int table_stride,
                 const int* __restrict__ positions, const int* __restrict__ row_entry, int nQ, int nK, int nV, int d,
                 int dv, int page_size, int num_pages, float eps, int* __restrict__ status, int whole, float temp_coef,
-                int temp_every, int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag) {
+                int temp_every, int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag, int v_norm, int v_mode,
+                float v_lambda, float* __restrict__ v_first) {
     extern __shared__ float rot[];                      // cos[rot_dims/2], sin[rot_dims/2]
     __shared__ float red[32];
     ng_pdl_trigger();
@@ -143,6 +148,31 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
     }
     if (page_ok) {
         const T* vs = in + (size_t)(v_is_k ? nQ : nQ + nK) * d;      // v_is_k: the values are the keys as projected
+        if (v_norm || v_mode) {                          // a warp per value head, float32 until the store
+            v_first = ng_after_wait(v_first);
+            for (int hv = blockIdx.y * MA_WARPS + warp; hv < nV; hv += MA_WARPS * gridDim.y) {
+                float v[2 * MA_DVU], ss = 0.f;
+#pragma unroll
+                for (int u = 0; u < 2 * MA_DVU; ++u) {
+                    const int c = lane + 32 * u;
+                    v[u] = c < dv ? ng_ld(vs + (size_t)hv * dv + c) : 0.f;
+                    ss += v[u] * v[u];
+                }
+                const float r = v_norm ? rsqrtf(ng_warp_sum(ss) / (float)dv + eps) : 1.f;
+                T* dst = v_pages + v_base + (size_t)hv * page_size * dv;
+#pragma unroll
+                for (int u = 0; u < 2 * MA_DVU; ++u) {
+                    const int c = lane + 32 * u;
+                    if (c >= dv) break;
+                    float y = v[u] * r;
+                    float* first = v_first + ((size_t)row * nV + hv) * dv + c;
+                    if (v_mode == 1) *first = y;
+                    else if (v_mode == 2) y = (1.f - v_lambda) * y + v_lambda * *first;
+                    ng_st(dst + c, y);
+                }
+            }
+            return;
+        }
         for (int j = blockIdx.y * MA_THREADS + threadIdx.x; j < nV * dv; j += MA_THREADS * gridDim.y) {
             const int hv = j / dv, c = j - hv * dv;
             v_pages[v_base + (size_t)hv * page_size * dv + c] = vs[j];
@@ -154,12 +184,13 @@ NG_EXPORT int ng_qkv_prep(const void* qkv, void* q_out, const float* qw, const f
                           int rot_dims, void* k_pages, void* v_pages, const int* table, int table_stride,
                           const int* positions, const int* row_entry, int n_rows, int nQ, int nK, int nV, int d, int dv,
                           int page_size, int num_pages, float eps, int* status, int whole, float temp_coef, int temp_every,
-                          int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag, int act_bf16,
-                          cudaStream_t stream) {
+                          int ld, int half_pairing, int unit_norm, int v_is_k, float rot_mag, int v_norm, int v_mode,
+                          float v_lambda, float* v_first, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (temp_every < 1 || (whole && (!qw || (nK > 0 && !kw)))) return NG_BAD_SIZE;
     if (ld < (nQ + nK) * d + (v_is_k ? 0 : nV * dv) || (unit_norm && (whole || qw || kw || rot_mag != 1.f)) ||
-        (v_is_k && (nV != nK || dv != d)))
+        (v_is_k && (nV != nK || dv != d)) || v_mode < 0 || v_mode > 2 || (v_mode && !v_first) ||
+        ((v_norm || v_mode) && dv > 64 * MA_DVU))
         return NG_BAD_SIZE;
     if (d <= 0 || d > 64 * MA_MAX_PAIRS || dv <= 0 || nQ <= 0 || nK < 0 || nV < 0 || page_size <= 0 || rot_dims < 0 ||
         rot_dims > d || (rot_dims & 1) || (rot_dims > 0 && !inv_freq))
@@ -171,11 +202,11 @@ NG_EXPORT int ng_qkv_prep(const void* qkv, void* q_out, const float* qw, const f
         NG_LAUNCH((qkv_prep_kernel<__nv_bfloat16>), grid, MA_THREADS, smem, stream, (const __nv_bfloat16*)qkv,
                   (__nv_bfloat16*)q_out, qw, kw, inv_freq, rot_dims, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, table,
                   table_stride, positions, row_entry, nQ, nK, nV, d, dv, page_size, num_pages, eps, status, whole, temp_coef,
-                  temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag);
+                  temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag, v_norm, v_mode, v_lambda, v_first);
     else
         NG_LAUNCH((qkv_prep_kernel<float>), grid, MA_THREADS, smem, stream, (const float*)qkv, (float*)q_out, qw, kw,
                   inv_freq, rot_dims, (float*)k_pages, (float*)v_pages, table, table_stride, positions, row_entry, nQ, nK, nV,
-                  d, dv, page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag);
+                  d, dv, page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag, v_norm, v_mode, v_lambda, v_first);
     return ng_launch_status();
 }
 
@@ -186,7 +217,17 @@ struct MaParams {
     int nH, nG, d, dv, page_size, num_pages, window, keep_first, n_splits, chunk;
     float scale, softcap, lambda, post_scale, eps; int head_norm;
     const float* slopes; const float* sinks;            // per head, or null
+    int sigmoid; const float* score_bias;               // weights sigmoid(s + score_bias[head]), not normalised
+    const void* gate; int gate_ld;                      // a logit per row and head whose sigmoid multiplies the head, or null
 };
+
+// what the last step multiplies a finished head by, besides its own norm
+template <typename T>
+__device__ __forceinline__ float ma_head_factor(const MaParams& p, int row, int head) {
+    float r = p.post_scale;
+    if (p.gate) r *= 1.f / (1.f + expf(-ng_ld(reinterpret_cast<const T*>(ng_after_wait(p.gate)) + (size_t)row * p.gate_ld + head)));
+    return r;
+}
 
 // the two bfloat16 values of a 32-bit word as float32: a bfloat16 is the upper half of a float32, so a shift and a
 // mask do it on the integer units (no conversion instruction)
@@ -240,7 +281,7 @@ __device__ __forceinline__ float2 ma_ld_pair(const float* v, int c, int dv, bool
 // sum_j p_j v_j,c (not yet divided by `l`), for the columns c = threadIdx.x, + MA_THREADS, ...
 template <typename T, int M>
 __device__ __forceinline__ void ma_finish(const MaParams& p, T* o, const float* acc /*[M][dv]*/, const float* l,
-                                          float* red) {
+                                          float* red, float factor) {
     float inv[M];
 #pragma unroll
     for (int m = 0; m < M; ++m) inv[m] = l[m] > 0.f ? 1.f / l[m] : 0.f;
@@ -253,7 +294,7 @@ __device__ __forceinline__ void ma_finish(const MaParams& p, T* o, const float* 
         keep[n] = v;
         ss += v * v;
     }
-    float r = p.post_scale;
+    float r = factor;
     if (p.head_norm) r *= rsqrtf(ng_block_sum(ss, red) / (float)p.dv + p.eps);
     n = 0;
     for (int c = threadIdx.x; c < p.dv; c += MA_THREADS, ++n) ng_st(o + c, keep[n] * r);
@@ -288,6 +329,7 @@ mapped_attention_kernel(const MaParams p) {
     __syncthreads();
     const int g = head / (p.nH / p.nG);
     const float slope = p.slopes ? p.slopes[head] : 0.f;
+    const float score_bias = p.sigmoid && p.score_bias ? p.score_bias[head] : 0.f;
     int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
     if (p.chunk > 0) lo = max(lo, (pos / p.chunk) * p.chunk);      // chunks count from the sequence's position 0
     const int n_sink = min(p.keep_first, lo);
@@ -306,7 +348,7 @@ mapped_attention_kernel(const MaParams p) {
     float m_run[M], l_run[M], acc[M][DVU][2];
 #pragma unroll
     for (int m = 0; m < M; ++m) {
-        m_run[m] = -INFINITY; l_run[m] = 0.f;
+        m_run[m] = p.sigmoid ? 0.f : -INFINITY; l_run[m] = 0.f;        // (sigmoid: no running maximum, every state counts whole)
 #pragma unroll
         for (int u = 0; u < DVU; ++u) acc[m][u][0] = acc[m][u][1] = 0.f;
     }
@@ -327,6 +369,10 @@ mapped_attention_kernel(const MaParams p) {
                 s = ma_dot(kp + kbase, q_s + m * d4, d, kvec) * p.scale;
                 if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
                 s -= slope * (float)(pos - kpos);
+            }
+            if (p.sigmoid) {
+                pr[m] = ok ? 1.f / (1.f + expf(-(s + score_bias))) : 0.f;
+                continue;
             }
             const float m_new = fmaxf(m_run[m], ng_warp_max(s));
             const float corr = m_run[m] == -INFINITY ? 0.f : expf(m_run[m] - m_new);
@@ -423,8 +469,8 @@ mapped_attention_kernel(const MaParams p) {
     __syncthreads();
     float lf[M];
 #pragma unroll
-    for (int m = 0; m < M; ++m) lf[m] = fin_l[m] + (p.sinks ? expf(p.sinks[head] - mt[m]) : 0.f);
-    ma_finish<T, M>(p, o, acc_s, lf, red);
+    for (int m = 0; m < M; ++m) lf[m] = p.sigmoid ? 1.f : fin_l[m] + (p.sinks ? expf(p.sinks[head] - mt[m]) : 0.f);
+    ma_finish<T, M>(p, o, acc_s, lf, red, ma_head_factor<T>(p, row, head));
 }
 
 // the runs of a (row, head) merged in run order, then the same last step
@@ -459,7 +505,7 @@ mapped_attention_merge_kernel(const MaParams p) {
             if (threadIdx.x < 32) f_s[s] = f;
             lt += ps[1] * f;
         }
-        lf[m] = ng_warp_sum(lt) + (p.sinks ? expf(p.sinks[head] - mt) : 0.f);
+        lf[m] = p.sigmoid ? 1.f : ng_warp_sum(lt) + (p.sinks ? expf(p.sinks[head] - mt) : 0.f);
         __syncthreads();
         for (int c = threadIdx.x; c < dv; c += MA_THREADS) {
             float a = 0.f;
@@ -469,7 +515,7 @@ mapped_attention_merge_kernel(const MaParams p) {
         }
     }
     __syncthreads();
-    ma_finish<T, M>(p, o, sm, lf, red);
+    ma_finish<T, M>(p, o, sm, lf, red, ma_head_factor<T>(p, row, head));
 }
 
 template <typename T, int M>
@@ -494,30 +540,35 @@ NG_EXPORT int ng_mapped_attention(const void* q, const void* k_pages, const void
                                   float* partial, int n_rows, int nH, int nG, int n_maps, int d, int dv, int page_size,
                                   int num_pages, int window, int keep_first, int n_splits, float scale, float softcap,
                                   float lambda, float post_scale, float eps, int head_norm, const float* slopes,
-                                  const float* sinks, int chunk, int act_bf16, cudaStream_t stream) {
+                                  const float* sinks, int chunk, int sigmoid, const float* score_bias, const void* gate,
+                                  int gate_ld, int act_bf16, cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (d <= 0 || dv <= 0 || dv > 64 * MA_DVU || nH <= 0 || nG <= 0 || nH % nG || page_size <= 0 || n_maps < 1 ||
         n_maps > 2 || n_splits < 1 || n_splits > 65535 || nH > 65535 || (n_splits > 1 && !partial) || out_ld < nH * dv ||
-        window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0))
+        window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0) ||
+        (sigmoid && (n_maps != 1 || sinks)) || (gate && gate_ld < nH))
         return NG_BAD_SIZE;
     MaParams p{q, k_pages, v_pages, table, table_stride, positions, row_entry, out, out_ld, n_splits > 1 ? partial : nullptr,
                nH, nG, d, dv, page_size, num_pages, window, keep_first, n_splits, chunk, scale, softcap, lambda, post_scale, eps,
-               head_norm, slopes, sinks};
+               head_norm, slopes, sinks, sigmoid, score_bias, gate, gate_ld};
     if (act_bf16) return n_maps == 2 ? ma_launch<__nv_bfloat16, 2>(p, n_rows, stream) : ma_launch<__nv_bfloat16, 1>(p, n_rows, stream);
     return n_maps == 2 ? ma_launch<float, 2>(p, n_rows, stream) : ma_launch<float, 1>(p, n_rows, stream);
 }
 
 // The runs' states of every (row, head) merged and the heads finished (maps combined, head norm), for states that another
 // kernel left in `partial` (float32 [n_rows, nH, n_splits, n_maps, dv + 2]: maximum, sum, weighted values).  Rows of no
-// entry get zeros.  `sinks` (per head, or null) adds exp(sink) to every head's sum.
+// entry get zeros.  `sinks` (per head, or null) adds exp(sink) to every head's sum.  `sigmoid`: the weights are not
+// normalised (the states' maxima are 0 and their sums not read); `gate` as above.
 NG_EXPORT int ng_mapped_attention_merge(float* partial, const int* row_entry, void* out, int out_ld, int n_rows, int nH,
                                         int n_maps, int dv, int n_splits, float lambda, float post_scale, float eps,
-                                        int head_norm, const float* sinks, int act_bf16, cudaStream_t stream) {
+                                        int head_norm, const float* sinks, int sigmoid, const void* gate, int gate_ld, int act_bf16,
+                                        cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
-    if (!partial || dv <= 0 || dv > 64 * MA_DVU || nH <= 0 || nH > 65535 || n_maps < 1 || n_maps > 2 || n_splits < 1 || out_ld < nH * dv)
+    if (!partial || dv <= 0 || dv > 64 * MA_DVU || nH <= 0 || nH > 65535 || n_maps < 1 || n_maps > 2 || n_splits < 1 || out_ld < nH * dv ||
+        (sigmoid && (n_maps != 1 || sinks)) || (gate && gate_ld < nH))
         return NG_BAD_SIZE;
     MaParams p{nullptr, nullptr, nullptr, nullptr, 0, nullptr, row_entry, out, out_ld, partial, nH, 1, 0, dv, 1, 0, 0, 0, n_splits, 0,
-               0.f, 0.f, lambda, post_scale, eps, head_norm, nullptr, sinks};
+               0.f, 0.f, lambda, post_scale, eps, head_norm, nullptr, sinks, sigmoid, nullptr, gate, gate_ld};
     dim3 grid(n_rows, nH);
     const size_t smem = ((size_t)n_maps * dv + n_splits) * sizeof(float);
     if (smem > 48 * 1024) return NG_BAD_SIZE;

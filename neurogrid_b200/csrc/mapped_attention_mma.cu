@@ -12,7 +12,9 @@
 // tokens then the window, in tiles of 64: keys (of each map) and values are staged once in shared memory for the four
 // warps (16-byte asynchronous copies through the block table, a tile ahead of the one being worked on), S = Q K^T in registers, mask and cap per element,
 // P V with P straight from the accumulators' layout, values through ldmatrix.trans.  Specialised on the key and
-// value sizes (-DNG_MA_D, -DNG_MA_DV: multiples of 16, up to 128).
+// value sizes (-DNG_MA_D, -DNG_MA_DV: multiples of 16, up to 128).  -DNG_MA_SIGMOID=1 builds the form without softmax (one
+// map): a visible key's weight is sigmoid(score + score_bias[head]), nothing is normalised, no maximum is kept.  `gate`
+// (optional): a logit per row and head whose sigmoid multiplies the finished head.
 #include "ng_common.cuh"
 
 #if !defined(NG_MA_D) || !defined(NG_MA_DV)
@@ -20,6 +22,11 @@
 #endif
 static_assert(NG_MA_D % 16 == 0 && NG_MA_D >= 16 && NG_MA_D <= 128, "key size: a multiple of 16 up to 128");
 static_assert(NG_MA_DV % 16 == 0 && NG_MA_DV >= 16 && NG_MA_DV <= 128, "value size: a multiple of 16 up to 128");
+
+#ifndef NG_MA_SIGMOID
+#define NG_MA_SIGMOID 0
+#endif
+constexpr bool SIGMOID = NG_MA_SIGMOID != 0;
 
 typedef __nv_bfloat16 bf16;
 constexpr int D = NG_MA_D, DV = NG_MA_DV;
@@ -35,6 +42,8 @@ struct MmaParams {
     float scale, softcap, lambda, post_scale, eps; int head_norm;
     float* partial; int n_splits;      // GROUP: runs of keys, their states [row, head, run, map, DV + 2]
     const float* slopes; const float* sinks;    // per head or null: slope * (pos - key position) off every score; exp(sink) in the sum
+    const float* score_bias;           // SIGMOID: added to head h's scores, or null
+    const bf16* gate; int gate_ld;     // a logit per row and head, rows gate_ld apart, or null
 };
 
 __device__ __forceinline__ void ldsm_x4(uint32_t (&r)[4], const void* p) {
@@ -62,6 +71,12 @@ __device__ __forceinline__ void cp_async16(void* dst, const void* src, bool real
 __device__ __forceinline__ float ex2f(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+// 1 / x on the special-function unit (relative error about 2^-23; 1 / inf = 0)
+__device__ __forceinline__ float rcpf(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 // tanh(x) = 1 - 2 / (1 + e^(2x)): exact limits at both ends, absolute error of a few 1e-7
@@ -161,10 +176,15 @@ mapped_attention_mma_kernel(const MmaParams p) {
         slope_a = p.slopes[GROUP ? head + min(row_a, n_rows - 1) : head] * 1.4426950408889634f;
         slope_b = p.slopes[GROUP ? head + min(row_b, n_rows - 1) : head] * 1.4426950408889634f;
     }
+    float sb_a = 0.f, sb_b = 0.f;                        // SIGMOID: the scores' bias, the same way
+    if (SIGMOID && p.score_bias) {
+        sb_a = p.score_bias[GROUP ? head + min(row_a, n_rows - 1) : head] * 1.4426950408889634f;
+        sb_b = p.score_bias[GROUP ? head + min(row_b, n_rows - 1) : head] * 1.4426950408889634f;
+    }
     float o[DV / 8][4];
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j) o[j][0] = o[j][1] = o[j][2] = o[j][3] = 0.f;
-    float m_a = -INFINITY, m_b = -INFINITY, l_a = 0.f, l_b = 0.f;
+    float m_a = SIGMOID ? 0.f : -INFINITY, m_b = m_a, l_a = 0.f, l_b = 0.f;
     const int* trow = p.table + (size_t)entry * p.table_stride;
 
     // Two buffers: while the warps work on a tile, the next one is on its way (cp.async, 16 bytes a copy; a key that
@@ -281,6 +301,13 @@ mapped_attention_mma_kernel(const MmaParams p) {
                 if (e < 2) mx_a = fmaxf(mx_a, v); else mx_b = fmaxf(mx_b, v);
             }
         }
+        if (SIGMOID) {                                   // 1 / (1 + 2^-t): a key the mask hides has t = -inf and weighs 0
+#pragma unroll
+            for (int j = 0; j < KW / 8; ++j) {
+                s[j][0] = rcpf(1.f + ex2f(-(s[j][0] + sb_a))); s[j][1] = rcpf(1.f + ex2f(-(s[j][1] + sb_a)));
+                s[j][2] = rcpf(1.f + ex2f(-(s[j][2] + sb_b))); s[j][3] = rcpf(1.f + ex2f(-(s[j][3] + sb_b)));
+            }
+        } else {
         mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 1));
         mx_a = fmaxf(mx_a, __shfl_xor_sync(0xffffffffu, mx_a, 2));
         mx_b = fmaxf(mx_b, __shfl_xor_sync(0xffffffffu, mx_b, 1));
@@ -298,6 +325,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
             s[j][2] = ex2f(s[j][2] - ub); s[j][3] = ex2f(s[j][3] - ub);
             l_a += s[j][0] + s[j][1];
             l_b += s[j][2] + s[j][3];
+        }
         }
         // ---- O += P V, P as three bfloat16 terms
 #pragma unroll
@@ -376,7 +404,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
         if (m_a != -INFINITY) l_a += ex2f(sk - m_a);
         if (m_b != -INFINITY) l_b += ex2f(sk - m_b);
     }
-    const float ia = l_a > 0.f ? 1.f / l_a : 0.f, ib = l_b > 0.f ? 1.f / l_b : 0.f;
+    const float ia = SIGMOID ? 1.f : l_a > 0.f ? 1.f / l_a : 0.f, ib = SIGMOID ? 1.f : l_b > 0.f ? 1.f / l_b : 0.f;
 #pragma unroll
     for (int j = 0; j < DV / 8; ++j) {
         float* oa = Os + ((size_t)map * ROWS + row_a) * DV + j * 8 + 2 * tq;
@@ -385,6 +413,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
         ob[0] = o[j][2] * ib; ob[1] = o[j][3] * ib;
     }
     __syncthreads();
+    const bf16* gate = ng_after_wait(p.gate);
     for (int row = warp; row < n_rows; row += WARPS) {
         float v[DV / 32 + 1];
         float ss = 0.f;
@@ -399,6 +428,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
             }
         }
         float r = p.post_scale;
+        if (p.gate) r *= rcpf(1.f + ex2f(-1.4426950408889634f * __bfloat162float(gate[(size_t)(q0 + r0 + row) * p.gate_ld + head])));
         if (p.head_norm) r *= rsqrtf(ng_warp_sum(ss) / (float)DV + p.eps);
         bf16* dst = p.out + (size_t)(q0 + r0 + row) * p.out_ld + (size_t)head * DV;
 #pragma unroll
@@ -434,16 +464,21 @@ NG_EXPORT int ng_mapped_attention_mma(const void* q, const void* k_pages, const 
                                       int n_entries, int max_q, int nH, int nG, int n_maps, int d, int dv, int page_size,
                                       int num_pages, int window, int keep_first, float scale, float softcap, float lambda,
                                       float post_scale, float eps, int head_norm, const float* slopes, const float* sinks,
-                                      int chunk, cudaStream_t stream) {
+                                      int chunk, int sigmoid, const float* score_bias, const void* gate, int gate_ld,
+                                      cudaStream_t stream) {
     if (n_entries <= 0 || max_q <= 0) return NG_OK;
     if (d != D || dv != DV || nH <= 0 || nG <= 0 || nH % nG || page_size <= 0 || n_maps < 1 || n_maps > 2 || out_ld < nH * dv ||
         window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0) || ((uintptr_t)q & 15) ||
-        ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15))
+        ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || (sigmoid != 0) != SIGMOID || (SIGMOID && (n_maps != 1 || sinks)) ||
+        (gate && gate_ld < nH))
         return NG_BAD_SIZE;
     MmaParams p{(const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, table, table_stride, cu_q, ctx_before, (bf16*)out,
                 out_ld, nH, nG, page_size, num_pages, window, keep_first, chunk, scale, softcap, lambda, post_scale, eps, head_norm,
-                nullptr, 1, slopes, sinks};
-    return n_maps == 2 ? mma_launch<2, false>(p, n_entries, max_q, stream) : mma_launch<1, false>(p, n_entries, max_q, stream);
+                nullptr, 1, slopes, sinks, score_bias, (const bf16*)gate, gate_ld};
+#if !NG_MA_SIGMOID
+    if (n_maps == 2) return mma_launch<2, false>(p, n_entries, max_q, stream);
+#endif
+    return mma_launch<1, false>(p, n_entries, max_q, stream);
 }
 
 // The same for entries of one token: the heads of a KV group are the rows of a tile (nH / nG <= 16), every row's keys are
@@ -454,15 +489,19 @@ NG_EXPORT int ng_mapped_attention_group(const void* q, const void* k_pages, cons
                                         int table_stride, const int* cu_q, const int* ctx_before, float* partial,
                                         int n_entries, int n_splits, int nH, int nG, int n_maps, int d, int dv, int page_size,
                                         int num_pages, int window, int keep_first, float scale, float softcap,
-                                        const float* slopes, int chunk, cudaStream_t stream) {
+                                        const float* slopes, int chunk, int sigmoid, const float* score_bias,
+                                        cudaStream_t stream) {
     if (n_entries <= 0) return NG_OK;
     if (d != D || dv != DV || nH <= 0 || nG <= 0 || nH % nG || nH / nG > 16 || page_size <= 0 || n_maps < 1 || n_maps > 2 ||
         window < 0 || keep_first < 0 || chunk < 0 || (chunk > 0 && keep_first > 0) || n_splits < 1 || n_splits > 65535 || !partial ||
         ((uintptr_t)q & 15) ||
-        ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15))
+        ((uintptr_t)k_pages & 15) || ((uintptr_t)v_pages & 15) || (sigmoid != 0) != SIGMOID || (SIGMOID && n_maps != 1))
         return NG_BAD_SIZE;
     MmaParams p{(const bf16*)q, (const bf16*)k_pages, (const bf16*)v_pages, table, table_stride, cu_q, ctx_before, nullptr, 0,
                 nH, nG, page_size, num_pages, window, keep_first, chunk, scale, softcap, 0.f, 1.f, 0.f, 0, partial, n_splits, slopes,
-                nullptr};
-    return n_maps == 2 ? mma_launch<2, true>(p, n_entries, 1, stream) : mma_launch<1, true>(p, n_entries, 1, stream);
+                nullptr, score_bias, nullptr, 0};
+#if !NG_MA_SIGMOID
+    if (n_maps == 2) return mma_launch<2, true>(p, n_entries, 1, stream);
+#endif
+    return mma_launch<1, true>(p, n_entries, 1, stream);
 }

@@ -187,11 +187,14 @@ NG_EXPORT int ng_moe_scale(void* act, const float* weights, int n_rows, int E, i
 //   not use; with `wsg` (float32 [H]) column E receives sigmoid(wsg . x), the gate of a shared expert.
 //   `softmax_scores`: s = softmax(W_r x) over all experts instead of the sigmoid.  `group_max`: a group's score is its
 //   largest choice score.  `route_scale` multiplies the weights.
+//   `n_identity`: the last that many of the E experts are the identity; they take part in scores, choice and sum like the
+//   others but have no column of their own, the sum of their weights goes to one column behind the others (and behind the
+//   shared expert's gate, if there is one).
 template <typename T>
 __global__ void __launch_bounds__(512)
 moe_router_sigmoid_kernel(const T* __restrict__ x, const float* __restrict__ wr, const float* __restrict__ corr,
                           const float* __restrict__ wsg, float* __restrict__ weights, int H, int E, int ldw, int top_k,
-                          int n_groups, int keep_groups, int softmax_scores, int group_max, float route_scale) {
+                          int n_groups, int keep_groups, int softmax_scores, int group_max, float route_scale, int n_identity) {
     extern __shared__ float z[];               // [E] scores s, [E] choice scores, [n_groups] group scores
     float* choice = z + E;
     float* gscore = choice + E;
@@ -201,6 +204,7 @@ moe_router_sigmoid_kernel(const T* __restrict__ x, const float* __restrict__ wr,
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarp = blockDim.x >> 5;
     const T* xr = x + (size_t)row * H;
     float* out = weights + (size_t)row * ldw;
+    const int n_own = E - n_identity;          // experts with a column
     for (int e = warp; e < E + (wsg ? 1 : 0); e += nwarp) {
         const float* w = e < E ? wr + (size_t)e * H : wsg;
         float acc = 0.f;
@@ -216,8 +220,8 @@ moe_router_sigmoid_kernel(const T* __restrict__ x, const float* __restrict__ wr,
         acc = ng_warp_sum(acc);
         if (lane == 0) {
             const float s = 1.f / (1.f + expf(-acc));
-            if (e < E) { z[e] = softmax_scores ? acc : s; choice[e] = s + (corr ? corr[e] : 0.f); out[e] = 0.f; }
-            else out[E] = s;
+            if (e < E) { z[e] = softmax_scores ? acc : s; choice[e] = s + (corr ? corr[e] : 0.f); if (e < n_own) out[e] = 0.f; }
+            else out[n_own] = s;
         }
     }
     __syncthreads();
@@ -273,25 +277,33 @@ moe_router_sigmoid_kernel(const T* __restrict__ x, const float* __restrict__ wr,
             idx[k] = best;
             sum += z[best];
         }
-        for (int k = 0; k < top_k; ++k) out[idx[k]] = z[idx[k]] / (sum + 1e-20f) * route_scale;
+        float identity = 0.f;
+        for (int k = 0; k < top_k; ++k) {
+            const float w = z[idx[k]] / (sum + 1e-20f) * route_scale;
+            if (idx[k] < n_own) out[idx[k]] = w;
+            else identity += w;
+        }
+        if (n_identity) out[n_own + (wsg ? 1 : 0)] = identity;
     }
 }
 
 NG_EXPORT int ng_moe_router_sigmoid(const void* x, const float* wr, const float* corr, const float* wsg, float* weights,
                                     int n_rows, int H, int E, int ldw, int top_k, int n_groups, int keep_groups,
-                                    int softmax_scores, int group_max, float route_scale, int act_bf16, cudaStream_t stream) {
+                                    int softmax_scores, int group_max, float route_scale, int n_identity, int act_bf16,
+                                    cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
     if (H <= 0 || E <= 0 || top_k < 1 || top_k > E || top_k > MOE_MAX_TOP || E > 4096 || n_groups < 1 || E % n_groups ||
-        keep_groups < 1 || keep_groups > n_groups || top_k > keep_groups * (E / n_groups) || ldw < E + (wsg ? 1 : 0))
+        keep_groups < 1 || keep_groups > n_groups || top_k > keep_groups * (E / n_groups) || n_identity < 0 || n_identity > E ||
+        ldw < E - n_identity + (wsg ? 1 : 0) + (n_identity ? 1 : 0))
         return NG_BAD_SIZE;
     const size_t smem = (size_t)(2 * E + n_groups) * sizeof(float);
     const int threads = n_rows <= 64 ? 32 * (E < 4 ? 4 : E > 16 ? 16 : E) : 128;
     if (act_bf16)
         NG_LAUNCH((moe_router_sigmoid_kernel<__nv_bfloat16>), n_rows, threads, smem, stream, (const __nv_bfloat16*)x, wr, corr,
-                  wsg, weights, H, E, ldw, top_k, n_groups, keep_groups, softmax_scores, group_max, route_scale);
+                  wsg, weights, H, E, ldw, top_k, n_groups, keep_groups, softmax_scores, group_max, route_scale, n_identity);
     else
         NG_LAUNCH((moe_router_sigmoid_kernel<float>), n_rows, threads, smem, stream, (const float*)x, wr, corr, wsg, weights, H,
-                  E, ldw, top_k, n_groups, keep_groups, softmax_scores, group_max, route_scale);
+                  E, ldw, top_k, n_groups, keep_groups, softmax_scores, group_max, route_scale, n_identity);
     return ng_launch_status();
 }
 
@@ -328,5 +340,33 @@ NG_EXPORT int ng_moe_clamped_glu_scaled(const void* gate_up, const float* weight
     else
         NG_LAUNCH((moe_clamped_glu_scaled_kernel<float>), grid, 256, 0, stream, (const float*)gate_up, weights, ldw,
                   (float*)out, I, E, ff, limit_e, limit_s, alpha, shared_gated);
+    return ng_launch_status();
+}
+
+// moe_identity_add: y[row, c] += weights[row] * x[row, c] with `weights` rows ldw apart (the column of the identity experts),
+//   x of the activation type; y is float32 (the stream, or a partial sum) or of the activation type.
+template <typename T, typename TY>
+__global__ void moe_identity_add_kernel(TY* __restrict__ y, const T* __restrict__ x, const float* __restrict__ weights, int ldw, int H) {
+    ng_pdl_trigger();
+    ng_pdl_wait();
+    const int row = blockIdx.y;
+    const int c = blockIdx.x * blockDim.x + threadIdx.x;
+    if (c >= H) return;
+    TY* p = y + (size_t)row * H + c;
+    ng_st(p, fmaf(weights[(size_t)row * ldw], ng_ld(x + (size_t)row * H + c), ng_ld(p)));
+}
+
+NG_EXPORT int ng_moe_identity_add(void* y, const void* x, const float* weights, int ldw, int n_rows, int H, int y_f32, int act_bf16,
+                                  cudaStream_t stream) {
+    if (n_rows <= 0) return NG_OK;
+    if (H <= 0 || ldw < 1 || n_rows > 65535) return NG_BAD_SIZE;
+    dim3 grid((H + 255) / 256, n_rows);
+    if (act_bf16 && y_f32)
+        NG_LAUNCH((moe_identity_add_kernel<__nv_bfloat16, float>), grid, 256, 0, stream, (float*)y, (const __nv_bfloat16*)x, weights, ldw, H);
+    else if (act_bf16)
+        NG_LAUNCH((moe_identity_add_kernel<__nv_bfloat16, __nv_bfloat16>), grid, 256, 0, stream, (__nv_bfloat16*)y,
+                  (const __nv_bfloat16*)x, weights, ldw, H);
+    else
+        NG_LAUNCH((moe_identity_add_kernel<float, float>), grid, 256, 0, stream, (float*)y, (const float*)x, weights, ldw, H);
     return ng_launch_status();
 }

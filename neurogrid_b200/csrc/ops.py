@@ -10,7 +10,7 @@ from __future__ import annotations
 
 import ctypes
 import os
-from typing import Optional
+from typing import Optional, Tuple
 
 import torch
 
@@ -406,7 +406,8 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
              table: torch.Tensor, positions: torch.Tensor, row_entry: torch.Tensor, n_q: int, n_k: int, n_v: int,
              dim: int, vdim: int, eps: float, status: torch.Tensor, *, whole: bool = False, q_temp_coef: float = 0.0,
              q_temp_every: int = 1, half_pairing: bool = False, unit_norm: bool = False, v_is_k: bool = False,
-             rot_mag: float = 1.0) -> None:
+             rot_mag: float = 1.0, v_norm: bool = False, v_first: Optional[torch.Tensor] = None,
+             v_lambda: Optional[float] = None) -> None:
     """qkv[N, (n_q + n_k) * dim + n_v * vdim]: every q and k head (a map of a head counts as one) gets its RMS norm
     over ``dim`` (if its weight is given; float32, shared by all heads) and the rotation of its first
     2 * len(inv_freq) coordinates in pairs (2i, 2i+1) by position * inv_freq[i]; q -> q_out[N, n_q * dim],
@@ -417,7 +418,8 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
     pair as (i, i + rot_dims/2).  ``unit_norm`` (without norm weights): every q and k head is divided by its root mean
     square all the same.  ``qkv`` may have further columns behind v; they are not read.  ``v_is_k``: there are no v columns,
     the values are the keys as projected (no norm, no rotation; n_v = n_k, vdim = dim).  ``rot_mag`` multiplies cosines
-    and sines."""
+    and sines.  ``v_norm``: every value head is divided by its root mean square.  ``v_first`` (float32 [N, n_v * vdim])
+    receives the values (``v_lambda`` None), or gives those that are mixed in: v <- (1 - v_lambda) v + v_lambda v_first."""
     n = q_out.shape[0]
     if q_out.shape != (n, n_q * dim) or qkv.dim() != 2 or qkv.shape[0] != n \
             or qkv.shape[1] < (n_q + n_k) * dim + (0 if v_is_k else n_v * vdim) or qkv.dtype != q_out.dtype \
@@ -434,18 +436,38 @@ def qkv_prep(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optional[torch.Te
     rot_dims = 2 * inv_freq.numel() if inv_freq is not None else 0
     if whole and (q_weight is None or q_weight.numel() != n_q * dim or (n_k and (k_weight is None or k_weight.numel() != n_k * dim))):
         raise KernelError("qkv_prep: a norm over the whole projection needs weights of the projection's length")
+    v_mode = 0 if v_first is None else 1 if v_lambda is None else 2
+    if (v_mode and (n_v == 0 or v_first.shape != (n, n_v * vdim))) or (v_lambda is not None and not v_mode):
+        raise KernelError("qkv_prep: mixed values are float32 [N, n_v * vdim]")
+    _f32(v_first, "first values")
     f = _fn("mapped_attention", "ng_qkv_prep", [_c_void_p] * 5 + [_c_int] + [_c_void_p] * 3 + [_c_int] + [_c_void_p] * 2
             + [_c_int] * 8 + [_c_float, _c_void_p, _c_int, _c_float, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int,
-                              _c_void_p])
+                              _c_int, _c_float, _c_void_p, _c_int, _c_void_p])
     _check(f(_ptr(qkv), _ptr(q_out), _ptr(q_weight), _ptr(k_weight), _ptr(inv_freq), rot_dims,
              _ptr(k_pages) if n_k else None, _ptr(v_pages) if n_v else None, _ptr(table), table.shape[1], _ptr(positions),
              _ptr(row_entry), n, n_q, n_k, n_v, dim, vdim, page_size, num_pages, float(eps), _ptr(status),
              int(bool(whole)), float(q_temp_coef), int(q_temp_every), qkv.shape[1], int(bool(half_pairing)),
-             int(bool(unit_norm)), int(bool(v_is_k)), float(rot_mag), _act_flag(q_out, "q_out"), _stream()), "qkv_prep")
+             int(bool(unit_norm)), int(bool(v_is_k)), float(rot_mag), int(bool(v_norm)), v_mode, float(v_lambda or 0.0),
+             _ptr(v_first), _act_flag(qkv, "qkv"), _stream()), "qkv_prep")
 
 
 def mapped_attention_partial_floats(n_rows: int, n_heads: int, n_maps: int, vdim: int, n_splits: int) -> int:
     return n_rows * n_heads * n_splits * n_maps * (vdim + 2) if n_splits > 1 else 0
+
+
+def _head_gate(gate: Optional[torch.Tensor], q: torch.Tensor, n_heads: int):
+    """(pointer, row pitch) of a gate's logits [N, n_heads] of the activation type, which may be columns of a wider buffer."""
+    if gate is None:
+        return None, 0
+    if gate.shape != (q.shape[0], n_heads) or gate.dtype != q.dtype:
+        raise KernelError("a gate per head has a logit of the activation type per row and head")
+    return gate.data_ptr(), max(_column_block(gate, "head gate"), n_heads)
+
+
+def _sigmoid_args(sigmoid: bool, score_bias: Optional[torch.Tensor], n_maps: int, sinks, n_heads: int):
+    if (sigmoid and (n_maps != 1 or sinks is not None)) or (score_bias is not None and not sigmoid):
+        raise KernelError("sigmoid weights have one map per head and no sink, and the scores' bias belongs to them")
+    return int(bool(sigmoid)), _slopes(score_bias, n_heads)
 
 
 def _post(head_norm: bool, post_scale: float, out_scale: float) -> float:
@@ -458,7 +480,8 @@ def mapped_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
                      window: Optional[int], keep_first: int, scale: float, softcap: float, lam: float, head_norm: bool,
                      post_scale: float, eps: float, n_splits: int = 1, partial: Optional[torch.Tensor] = None,
                      slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
-                     out_scale: float = 1.0) -> None:
+                     out_scale: float = 1.0, sigmoid: bool = False, score_bias: Optional[torch.Tensor] = None,
+                     gate: Optional[torch.Tensor] = None) -> None:
     """Attention with float32 scores and weights over keys [P, G * n_maps, page, dim] and values [P, G, page, vdim]:
     per head and map m, a_m = softmax(cap(scale * q_m . k_m)) v over the keys j <= pos with pos - j < window or
     j < keep_first (window None: all), cap(s) = softcap * tanh(s / softcap) (softcap 0: none); the head's output is
@@ -468,7 +491,9 @@ def mapped_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     ``mapped_attention_partial_floats`` values): for steps of few rows.  ``slopes`` (float32 [n_heads]): slope[head] *
     (position - key position) is taken off every score; ``sinks`` (float32 [n_heads]): every softmax's denominator
     also holds exp(sink[head]), a term that has no key and no value.  ``chunk`` > 0: a row also sees only the keys of
-    its own chunk, floor(j / chunk) = floor(pos / chunk)."""
+    its own chunk, floor(j / chunk) = floor(pos / chunk).  ``sigmoid`` (one map): no softmax, a visible key's weight is
+    sigmoid(score + score_bias[head]) (``score_bias`` float32 [n_heads] or None), not normalised over the keys.  ``gate``
+    [N, n_heads] (activation type, may be columns of a wider buffer): head h of row r times sigmoid(gate[r, h])."""
     n = q.shape[0]
     num_pages, n_k, page_size, dim = k_pages.shape
     n_g, vdim = v_pages.shape[1], v_pages.shape[3]
@@ -481,12 +506,15 @@ def mapped_attention(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tens
     if need and (partial is None or partial.numel() < need):
         raise KernelError(f"mapped_attention: the runs need {need} float32 values")
     f = _fn("mapped_attention", "ng_mapped_attention", [_c_void_p] * 4 + [_c_int] + [_c_void_p] * 3 + [_c_int, _c_void_p]
-            + [_c_int] * 11 + [_c_float] * 5 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p])
+            + [_c_int] * 11 + [_c_float] * 5 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int,
+                                                _c_void_p])
     _check(f(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], _ptr(positions), _ptr(row_entry),
              out.data_ptr(), _column_block(out, "attention out"), _ptr(partial) if need else None, n, n_heads, n_g, n_maps,
              dim, vdim, page_size, num_pages, int(window or 0), int(keep_first), int(n_splits), float(scale),
              float(softcap or 0.0), float(lam), _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)),
-             _slopes(slopes, n_heads), _slopes(sinks, n_heads), int(chunk or 0), _act_flag(q, "q"), _stream()), "mapped_attention")
+             _slopes(slopes, n_heads), _slopes(sinks, n_heads), int(chunk or 0),
+             *_sigmoid_args(sigmoid, score_bias, n_maps, sinks, n_heads), *_head_gate(gate, q, n_heads), _act_flag(q, "q"),
+             _stream()), "mapped_attention")
 
 
 MAPPED_BACKEND = os.environ.get("NEUROGRID_B200_MAPPED", "mma")     # "mma": tensor-core kernel for long bfloat16 steps; "ffma"
@@ -498,12 +526,18 @@ def mapped_attention_mma_takes(dim: int, vdim: int, dtype) -> bool:
         and 16 <= dim <= 128 and 16 <= vdim <= 128
 
 
+def mapped_attention_mma_defines(dim: int, vdim: int, sigmoid: bool = False):
+    """The tensor-core library's specialisation for these sizes and this kind of weights."""
+    return {"NG_MA_D": dim, "NG_MA_DV": vdim, **({"NG_MA_SIGMOID": 1} if sigmoid else {})}
+
+
 def mapped_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.Tensor, table: torch.Tensor,
                          cu_q: torch.Tensor, ctx_before: torch.Tensor, out: torch.Tensor, n_entries: int, max_q: int,
                          n_heads: int, n_maps: int, window: Optional[int], keep_first: int, scale: float, softcap: float,
                          lam: float, head_norm: bool, post_scale: float, eps: float,
                          slopes: Optional[torch.Tensor] = None, sinks: Optional[torch.Tensor] = None, chunk: int = 0,
-                     out_scale: float = 1.0) -> None:
+                         out_scale: float = 1.0, sigmoid: bool = False, score_bias: Optional[torch.Tensor] = None,
+                         gate: Optional[torch.Tensor] = None) -> None:
     """``mapped_attention`` for long bfloat16 steps on the tensor cores: scores are float32 sums of exact bfloat16
     products, the float32 softmax weights enter the weighted sum as three bfloat16 terms each.  Rows are named by
     ``cu_q`` [R+1] and ``ctx_before`` [R]; ``max_q`` bounds the longest entry."""
@@ -516,12 +550,14 @@ def mapped_attention_mma(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torch.
         raise KernelError("mapped_attention_mma: shapes or dtypes do not fit")
     _i32(table, "table"), _i32(cu_q, "cu_q"), _i32(ctx_before, "ctx_before")
     f = _fn("mapped_attention_mma", "ng_mapped_attention_mma", [_c_void_p] * 4 + [_c_int] + [_c_void_p] * 3 + [_c_int] * 12
-            + [_c_float] * 5 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_void_p], {"NG_MA_D": dim, "NG_MA_DV": vdim})
+            + [_c_float] * 5 + [_c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p],
+            mapped_attention_mma_defines(dim, vdim, sigmoid))
     _check(f(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], _ptr(cu_q), _ptr(ctx_before),
              out.data_ptr(), _column_block(out, "attention out"), n_entries, max_q, n_heads, n_g, n_maps, dim, vdim,
              page_size, num_pages, int(window or 0), int(keep_first), float(scale), float(softcap or 0.0), float(lam),
              _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)), _slopes(slopes, n_heads), _slopes(sinks, n_heads),
-             int(chunk or 0), _stream()), "mapped_attention_mma")
+             int(chunk or 0), *_sigmoid_args(sigmoid, score_bias, n_maps, sinks, n_heads), *_head_gate(gate, q, n_heads),
+             _stream()), "mapped_attention_mma")
 
 
 def mapped_attention_group_takes(dim: int, vdim: int, n_heads: int, n_kv_heads: int, dtype) -> bool:
@@ -534,7 +570,9 @@ def mapped_attention_group(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
                            partial: torch.Tensor, n_entries: int, n_heads: int, n_maps: int, window: Optional[int],
                            keep_first: int, scale: float, softcap: float, lam: float, head_norm: bool, post_scale: float,
                            eps: float, n_splits: int, slopes: Optional[torch.Tensor] = None,
-                           sinks: Optional[torch.Tensor] = None, chunk: int = 0, out_scale: float = 1.0) -> None:
+                           sinks: Optional[torch.Tensor] = None, chunk: int = 0, out_scale: float = 1.0,
+                           sigmoid: bool = False, score_bias: Optional[torch.Tensor] = None,
+                           gate: Optional[torch.Tensor] = None) -> None:
     """``mapped_attention`` for a step whose entries bring one token each (bfloat16), on the tensor cores: the query
     heads of a KV group are the rows of a tile, every row's keys are cut into ``n_splits`` runs (a block each), and the
     runs' states pass through ``partial`` (float32, ``mapped_attention_partial_floats`` values, also for one run) to
@@ -550,17 +588,19 @@ def mapped_attention_group(q: torch.Tensor, k_pages: torch.Tensor, v_pages: torc
     if partial is None or partial.dtype != torch.float32 or partial.numel() < need:
         raise KernelError(f"mapped_attention_group: the runs need {need} float32 values")
     _i32(table, "table"), _i32(cu_q, "cu_q"), _i32(ctx_before, "ctx_before"), _i32(row_entry, "row_entry")
-    defines = {"NG_MA_D": dim, "NG_MA_DV": vdim}
+    defines = mapped_attention_mma_defines(dim, vdim, sigmoid)
+    sig, bias = _sigmoid_args(sigmoid, score_bias, n_maps, sinks, n_heads)
     f = _fn("mapped_attention_mma", "ng_mapped_attention_group", [_c_void_p] * 4 + [_c_int] + [_c_void_p] * 3 + [_c_int] * 11
-            + [_c_float] * 2 + [_c_void_p, _c_int, _c_void_p], defines)
+            + [_c_float] * 2 + [_c_void_p, _c_int, _c_int, _c_void_p, _c_void_p], defines)
     _check(f(_ptr(q), _ptr(k_pages), _ptr(v_pages), _ptr(table), table.shape[1], _ptr(cu_q), _ptr(ctx_before), _ptr(partial),
              n_entries, int(n_splits), n_heads, n_g, n_maps, dim, vdim, page_size, num_pages, int(window or 0), int(keep_first),
-             float(scale), float(softcap or 0.0), _slopes(slopes, n_heads), int(chunk or 0), _stream()), "mapped_attention_group")
+             float(scale), float(softcap or 0.0), _slopes(slopes, n_heads), int(chunk or 0), sig, bias, _stream()),
+           "mapped_attention_group")
     g = _fn("mapped_attention", "ng_mapped_attention_merge", [_c_void_p] * 3 + [_c_int] * 6 + [_c_float] * 3
-            + [_c_int, _c_void_p, _c_int, _c_void_p])
+            + [_c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
     _check(g(_ptr(partial), _ptr(row_entry), out.data_ptr(), _column_block(out, "attention out"), n, n_heads, n_maps, vdim,
-             int(n_splits), float(lam), _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)), _slopes(sinks, n_heads), 1, _stream()),
-           "mapped_attention_merge")
+             int(n_splits), float(lam), _post(head_norm, post_scale, out_scale), float(eps), int(bool(head_norm)), _slopes(sinks, n_heads), sig,
+             *_head_gate(gate, q, n_heads), 1, _stream()), "mapped_attention_merge")
 
 
 # ----------------------------------------------------------------------------- input convolution
@@ -630,43 +670,44 @@ def retention_chunked_takes(key_dim: int, value_dim: int) -> bool:
 
 # ----------------------------------------------------------------------------- latent attention
 def latent_prep(x: torch.Tensor, wq: torch.Tensor, wkv: torch.Tensor, cq_out: torch.Tensor, pages: torch.Tensor,
-                gate_out: torch.Tensor, table: torch.Tensor, positions: torch.Tensor, row_entry: torch.Tensor,
+                gate_out: Optional[torch.Tensor], table: torch.Tensor, positions: torch.Tensor, row_entry: torch.Tensor,
                 n_heads: int, eps: float, status: torch.Tensor, *, rot: int = 0, inv_freq: Optional[torch.Tensor] = None,
-                half_pairing: bool = False) -> None:
+                half_pairing: bool = False, rot_mag: float = 1.0) -> None:
     """x[N, rq+rkv+rot+nH] = c_q raw | c raw | key part raw | gate logits;  cq_out[N, rq] = rmsnorm(c_q raw) * wq;
     rmsnorm(c raw) * wkv goes to the row's place in pages[P, 1, page, rp] and behind it the key part (``rot`` columns,
     not normed), rotated by the row's position in pairs (2i, 2i+1) or (i, i+rot/2) with ``inv_freq`` [rot/2]; the
-    columns behind are zero.  gate_out[N, nH] float32 = sigmoid(gate logits), nH the gate's columns.  ``wkv`` and
+    columns behind are zero.  gate_out[N, nH] float32 = sigmoid(gate logits), nH the gate's columns (0 with ``gate_out``
+    None: no gate).  ``rot_mag`` multiplies cosines and sines.  ``wkv`` and
     ``pages`` None: a layer that reads another layer's latents (the row has no c and no key part)."""
     n, rq = cq_out.shape
     rkv = wkv.numel() if wkv is not None else 0
     num_pages, one, page_size, rp = pages.shape if pages is not None else (0, 1, 1, 0)
     if x.shape != (n, rq + rkv + rot + n_heads) or wq.numel() != rq or one != 1 or rp < rkv + rot \
-            or gate_out.shape != (n, n_heads) or cq_out.dtype != x.dtype or (pages is not None and pages.dtype != x.dtype) \
+            or (gate_out is None) != (n_heads == 0) or (n_heads and gate_out.shape != (n, n_heads)) or cq_out.dtype != x.dtype or (pages is not None and pages.dtype != x.dtype) \
             or (rkv == 0) != (pages is None) or (rot and (inv_freq is None or inv_freq.numel() != rot // 2 or not rkv)):
         raise KernelError("latent_prep: shapes or dtypes do not fit")
     _f32(wq, "dq norm"), _f32(wkv, "dkv norm"), _f32(gate_out, "gate"), _f32(inv_freq, "inv_freq")
     _i32(table, "table"), _i32(positions, "positions"), _i32(row_entry, "row_entry"), _i32(status, "status")
     f = _fn("latent", "ng_latent_prep", [_c_void_p] * 7 + [_c_int] + [_c_void_p] * 2 + [_c_int] * 7
-            + [_c_float, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p])
+            + [_c_float, _c_void_p, _c_int, _c_void_p, _c_int, _c_float, _c_int, _c_void_p])
     _check(f(_ptr(x), _ptr(wq), _ptr(wkv), _ptr(cq_out), _ptr(pages), _ptr(gate_out), _ptr(table), table.shape[1],
              _ptr(positions), _ptr(row_entry), n, rq, rkv, rp, n_heads, page_size, num_pages, float(eps),
-             _ptr(status), int(rot), _ptr(inv_freq) if rot else None, int(bool(half_pairing)),
+             _ptr(status), int(rot), _ptr(inv_freq) if rot else None, int(bool(half_pairing)), float(rot_mag),
              _act_flag(x, "latent input"), _stream()), "latent_prep")
 
 
 def latent_rope_q(q: torch.Tensor, positions: torch.Tensor, row_entry: torch.Tensor, inv_freq: torch.Tensor,
-                  n_heads: int, offset: int, half_pairing: bool = False) -> None:
+                  n_heads: int, offset: int, half_pairing: bool = False, rot_mag: float = 1.0) -> None:
     """q[N, nH * rp]: columns offset..offset + 2 len(inv_freq) of every head are rotated in place by the row's position,
-    in pairs (2i, 2i+1) or (i, i + rot/2); angles float32."""
+    in pairs (2i, 2i+1) or (i, i + rot/2); angles float32, cosines and sines times ``rot_mag``."""
     n = q.shape[0]
     rp, rot = q.shape[1] // n_heads, 2 * inv_freq.numel()
     if q.shape[1] != n_heads * rp or offset + rot > rp:
         raise KernelError("latent_rope_q: shapes do not fit")
     _f32(inv_freq, "inv_freq"), _i32(positions, "positions"), _i32(row_entry, "row_entry")
-    f = _fn("latent", "ng_latent_rope_q", [_c_void_p] * 4 + [_c_int] * 7 + [_c_void_p])
+    f = _fn("latent", "ng_latent_rope_q", [_c_void_p] * 4 + [_c_int] * 6 + [_c_float, _c_int, _c_void_p])
     _check(f(_ptr(q), _ptr(positions), _ptr(row_entry), _ptr(inv_freq), n, n_heads, rp, int(offset), rot,
-             int(bool(half_pairing)), _act_flag(q, "q"), _stream()), "latent_rope_q")
+             int(bool(half_pairing)), float(rot_mag), _act_flag(q, "q"), _stream()), "latent_rope_q")
 
 
 def head_up_gate(o: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor) -> None:
@@ -895,14 +936,26 @@ def gate_mul(y: torch.Tensor, gate: Optional[torch.Tensor], activation: str = "s
              _stream()), "gate_mul")
 
 
+def _identity(identity, n: int, H: int, act_dtype):
+    """(pointer, pointer, pitch) of (z [N,H], w [N]): a multiple of each row of z is part of a sublayer's output."""
+    if identity is None:
+        return None, None, 0
+    z, w = identity
+    if z.shape != (n, H) or z.dtype != act_dtype or w.shape != (n,) or w.dtype != torch.float32 or not w.is_cuda:
+        raise KernelError("identity: z is [N, H] of the activation dtype, w float32 [N]")
+    return _ptr(z), w.data_ptr(), max(1, w.stride(0))
+
+
 def hc_step(streams: torch.Tensor, n_streams: int, *, x0: Optional[torch.Tensor] = None, delta: Optional[torch.Tensor] = None,
             mix: Optional[torch.Tensor] = None, out_w: Optional[torch.Tensor] = None, in_w: Optional[torch.Tensor] = None,
             norm_w: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-            sum_out: Optional[torch.Tensor] = None, eps: float = 0.0, act_dtype=None, bias: Optional[torch.Tensor] = None) -> None:
+            sum_out: Optional[torch.Tensor] = None, eps: float = 0.0, act_dtype=None, bias: Optional[torch.Tensor] = None,
+            identity: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> None:
     """What lies between two sublayers of a model whose residual stream is ``n_streams`` copies, streams[N, S * H]
     float32.  ``x0`` [N,H] float32: every copy is x0 (a sequence's start).  ``delta`` (the output y of the sublayer
     before: [N,H] of the activation dtype or a float32 stack of partial sums) with ``mix`` [S,S] ([from, to]) and
-    ``out_w`` [S]: x_t <- sum_s mix[s,t] x_s + out_w[t] y for all t at once (``bias`` [H] float32 belongs to y: it is added to it).  ``in_w`` [S] with ``norm_w`` [H] and
+    ``out_w`` [S]: x_t <- sum_s mix[s,t] x_s + out_w[t] y for all t at once (``bias`` [H] float32 belongs to y: it is added to it; so is
+    ``identity`` = (z [N,H] of the activation dtype, w [N] float32, may be a column of a wider buffer): y += w z).  ``in_w`` [S] with ``norm_w`` [H] and
     ``out`` [N,H]: out = rmsnorm(sum_t in_w[t] x_t) * norm_w.  ``sum_out`` [N,H] float32: the sum of the copies."""
     n = streams.shape[0]
     H = streams.shape[1] // n_streams
@@ -924,10 +977,11 @@ def hc_step(streams: torch.Tensor, n_streams: int, *, x0: Optional[torch.Tensor]
     for t in (x0, sum_out):
         if t is not None and t.shape != (n, H):
             raise KernelError("hc_step: x0 and sum_out are [N, H]")
-    f = _fn("hyper", "ng_hc_step", [_c_void_p] * 3 + [_c_int, _c_int, _c_ll] + [_c_void_p] * 7 + [_c_int] * 3
+    id_x, id_w, id_ld = _identity(identity, n, H, act_dtype)
+    f = _fn("hyper", "ng_hc_step", [_c_void_p] * 3 + [_c_int, _c_int, _c_ll] + [_c_void_p] * 9 + [_c_int] * 4
             + [_c_float, _c_int, _c_void_p])
     _check(f(_ptr(streams), _ptr(x0), _ptr(delta), d32, n_part, stride, _ptr(mix), _ptr(out_w), _ptr(in_w), _ptr(norm_w),
-             _ptr(out), _ptr(sum_out), _ptr(bias), n, int(n_streams), H, float(eps), act, _stream()), "hc_step")
+             _ptr(out), _ptr(sum_out), _ptr(bias), id_x, id_w, id_ld, n, int(n_streams), H, float(eps), act, _stream()), "hc_step")
 
 
 # ----------------------------------------------------------------------------- gated linear attention
@@ -1086,23 +1140,24 @@ def scale_(x: torch.Tensor, factor: float) -> None:
 def moe_router_sigmoid(x: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor],
                        w_shared_gate: Optional[torch.Tensor], weights: torch.Tensor, top_k: int, n_groups: int = 1,
                        keep_groups: int = 1, *, softmax_scores: bool = False, group_max: bool = False,
-                       route_scale: float = 1.0) -> None:
+                       route_scale: float = 1.0, n_identity: int = 0) -> None:
     """weights[N, E (+1)] float32: scores s = sigmoid(W_r x); the top_k experts by s + correction among the experts
     of the keep_groups best of n_groups groups of neighbours (a group's score: its two largest choice scores) get
     s / (sum of the chosen s + 1e-20), the others zero.  With ``w_shared_gate`` (float32 [H]) the last column
     receives sigmoid(w . x).  ``softmax_scores``: s = softmax(W_r x) over all experts instead; ``group_max``: a group's
-    score is its largest choice score; ``route_scale`` multiplies the weights."""
+    score is its largest choice score; ``route_scale`` multiplies the weights.  ``n_identity``: the last that many of the E
+    experts have no column; the sum of their weights goes to the last column (weights[N, E - n_identity (+1) + 1])."""
     n, H = x.shape
     E = w_router.shape[0]
     ldw = weights.shape[1]
-    if w_router.shape != (E, H) or weights.shape[0] != n or ldw != E + (w_shared_gate is not None) \
+    if w_router.shape != (E, H) or weights.shape[0] != n or ldw != E - n_identity + (w_shared_gate is not None) + (n_identity > 0) \
             or (correction is not None and correction.numel() != E) or (w_shared_gate is not None and w_shared_gate.numel() != H):
         raise KernelError("moe_router_sigmoid: shapes do not fit")
     _f32(w_router, "router weight"), _f32(correction, "correction"), _f32(w_shared_gate, "shared gate"), _f32(weights, "weights")
-    f = _fn("moe", "ng_moe_router_sigmoid", [_c_void_p] * 5 + [_c_int] * 9 + [_c_float, _c_int, _c_void_p])
+    f = _fn("moe", "ng_moe_router_sigmoid", [_c_void_p] * 5 + [_c_int] * 9 + [_c_float, _c_int, _c_int, _c_void_p])
     _check(f(_ptr(x), _ptr(w_router), _ptr(correction), _ptr(w_shared_gate), _ptr(weights), n, H, E, ldw, int(top_k),
              int(n_groups), int(keep_groups), int(bool(softmax_scores)), int(bool(group_max)), float(route_scale),
-             _act_flag(x, "router input"), _stream()), "moe_router_sigmoid")
+             int(n_identity), _act_flag(x, "router input"), _stream()), "moe_router_sigmoid")
 
 
 def moe_clamped_glu_scaled(gate_up: torch.Tensor, weights: torch.Tensor, out: torch.Tensor, n_experts: int, expert_ff: int,
@@ -1134,11 +1189,31 @@ def moe_router(x: torch.Tensor, w_router: torch.Tensor, b_router: Optional[torch
              _stream()), "moe_router")
 
 
-def moe_scale(act: torch.Tensor, weights: torch.Tensor, expert_ff: int, shared_gated: bool = False) -> None:
+def _moe_experts(weights, shared_gated, n_experts):
+    """Experts with a column of ``weights`` (None: all columns but the shared expert's gate)."""
+    E = weights.shape[1] - int(bool(shared_gated)) if n_experts is None else int(n_experts)
+    if weights.shape[1] < E + int(bool(shared_gated)):
+        raise KernelError("routing weights have a column per expert")
+    return E
+
+
+def moe_identity_add(y: torch.Tensor, x: torch.Tensor, w: torch.Tensor) -> None:
+    """y[N,H] += w[N] * x[N,H]: identity experts.  y float32 or of x's type; w float32, may be a column of a wider buffer."""
+    n, H = x.shape
+    if y.shape != (n, H) or y.dtype not in (torch.float32, x.dtype):
+        raise KernelError("moe_identity_add: shapes or dtypes do not fit")
+    px, pw, ld = _identity((x, w), n, H, x.dtype)
+    f = _fn("moe", "ng_moe_identity_add", [_c_void_p] * 3 + [_c_int] * 5 + [_c_void_p])
+    _check(f(_ptr(y), px, pw, ld, n, H, int(y.dtype == torch.float32), _act_flag(x, "moe input"), _stream()), "moe_identity_add")
+
+
+def moe_scale(act: torch.Tensor, weights: torch.Tensor, expert_ff: int, shared_gated: bool = False,
+              n_experts: Optional[int] = None) -> None:
     """act[N, ld]: columns e*ff..(e+1)*ff are multiplied by weights[N, e], in place; columns behind E*ff stay, or, with
-    ``shared_gated`` (weights then has a column E), are multiplied by weights[N, E]."""
+    ``shared_gated`` (weights then has a column E), are multiplied by weights[N, E].  ``n_experts``: E, when weights has
+    further columns."""
     n, ld = act.shape
-    E = weights.shape[1] - int(bool(shared_gated))
+    E = _moe_experts(weights, shared_gated, n_experts)
     if weights.shape[0] != n or ld < E * expert_ff:
         raise KernelError("moe_scale: shapes do not fit")
     _f32(weights, "routing weights")
@@ -1148,11 +1223,11 @@ def moe_scale(act: torch.Tensor, weights: torch.Tensor, expert_ff: int, shared_g
 
 
 def moe_swiglu_scaled(gate_up: torch.Tensor, weights: torch.Tensor, out: torch.Tensor, expert_ff: int,
-                      shared_gated: bool = False) -> None:
+                      shared_gated: bool = False, n_experts: Optional[int] = None) -> None:
     """out[N, I] = silu(gate_up[:, :I]) * gate_up[:, I:], columns e*ff..(e+1)*ff times weights[N, e] (float32); with
-    ``shared_gated`` the columns behind E*ff times weights[N, E]."""
+    ``shared_gated`` the columns behind E*ff times weights[N, E].  ``n_experts``: E, when weights has further columns."""
     n, I = out.shape
-    E = weights.shape[1] - int(bool(shared_gated))
+    E = _moe_experts(weights, shared_gated, n_experts)
     if gate_up.shape != (n, 2 * I) or gate_up.dtype != out.dtype or weights.shape[0] != n or I < E * expert_ff:
         raise KernelError("moe_swiglu_scaled: shapes do not fit")
     _f32(weights, "routing weights")
@@ -1278,18 +1353,21 @@ def gemm_splits(K: int, splits: int) -> int:
 
 
 def gemm_swiglu_sm100(x: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, *, token_tile: int = 0,
-                      activation: str = "silu", limit: float = 0.0, alpha: float = 0.0) -> None:
+                      activation: str = "silu", limit: float = 0.0, alpha: float = 0.0,
+                      bias: Optional[torch.Tensor] = None) -> None:
     """out[M,I] = act(x wg^T) * (x wu^T) with w_gate_up = [wg (I rows); wu (I rows)]: the gate is
-    applied in the product's epilogue (act = silu or the tanh form of gelu, or both halves clamped, as ``swiglu`` has them).  ``out`` may be a block of columns
-    of a wider buffer."""
+    applied in the product's epilogue (act = silu or the tanh form of gelu, or both halves clamped, as ``swiglu`` has them).  ``bias`` [2 I] (bfloat16) is
+    added to both products.  ``out`` may be a block of columns of a wider buffer."""
     M, K = x.shape
     I = out.shape[1]
+    if bias is not None and (bias.numel() != 2 * I or bias.dtype != torch.bfloat16):
+        raise KernelError("gemm_swiglu_sm100: the bias is bfloat16 [2 I]")
     if w_gate_up.shape != (2 * I, K) or out.shape[0] != M or out.dtype != torch.bfloat16 or activation not in GATE_ACTIVATIONS:
         raise KernelError("gemm_swiglu_sm100: shapes do not fit")
     ldc = _column_block(out, "gemm_swiglu_sm100 out")
     status = _ptr(_gemm_status(w_gate_up.device))
     f = _fn("gemm_sm100", "ng_gemm_sm100", _GEMM_ARGS)
-    _check(f(_ptr(x), _ptr(w_gate_up), None, out.data_ptr(), M, I, K, 2 * I, ldc,
+    _check(f(_ptr(x), _ptr(w_gate_up), _ptr(bias), out.data_ptr(), M, I, K, 2 * I, ldc,
              {"silu": 2, "gelu_tanh": 4, "clamped_glu": 6}[activation], 1, I, token_tile, float(limit), float(alpha), status, _stream()), "gemm_swiglu_sm100")
 
 

@@ -196,7 +196,7 @@ class Decoder:
             ops.hc_step(h, s.streams, sum_out=total, act_dtype=self.dtype)
         else:
             ops.hc_step(h, s.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, bias=pending.bias,
-                        sum_out=total, act_dtype=self.dtype)
+                        identity=pending.identity, sum_out=total, act_dtype=self.dtype)
         return total
 
     def finish(self, ctx: StepContext, h: torch.Tensor, pending, want_rows: Optional[torch.Tensor],

@@ -254,11 +254,11 @@ class ParallelBlock:
 
 class HyperPending:
     """What a hyper block leaves for the kernel after it: its last sublayer's output (not yet written into the copies of
-    the stream; ``bias``, float32 [H] or None, is still to be added to it) with the mixing matrix and output weights that
-    write it."""
+    the stream; ``bias``, float32 [H] or None, is still to be added to it, and so is ``identity``, (z [N,H], w [N]) or
+    None: w z) with the mixing matrix and output weights that write it."""
 
-    def __init__(self, y, mix, out_w, eps, bias=None):
-        self.y, self.mix, self.out_w, self.eps, self.bias = y, mix, out_w, eps, bias
+    def __init__(self, y, mix, out_w, eps, bias=None, identity=None):
+        self.y, self.mix, self.out_w, self.eps, self.bias, self.identity = y, mix, out_w, eps, bias, identity
 
 
 @register("block", "hyper")
@@ -294,8 +294,11 @@ class HyperBlock:
         self.mixer_norm = registry.build("norm", spec.mixer_norm, **kw)
         self.ffn_norm = registry.build("norm", spec.ffn_norm, **kw) if spec.ffn is not None else None
         self.hc = {}
-        if hasattr(self.mixer, "defer_bias"):                # its output's bias rides in the kernel behind it
-            self.mixer.defer_bias = True
+        for part in (self.mixer, self.ffn):
+            if hasattr(part, "defer_bias"):                  # its output's bias rides in the kernel behind it
+                part.defer_bias = True
+            if hasattr(part, "defer_identity"):              # ... and so does a multiple of what it read
+                part.defer_identity = True
 
     def parts(self):
         n = self.spec.names
@@ -352,7 +355,8 @@ class HyperBlock:
         elif pending is None:
             ops.hc_step(X, self.streams, **kw)
         else:
-            ops.hc_step(X, self.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, bias=pending.bias, **kw)
+            ops.hc_step(X, self.streams, delta=pending.y, mix=pending.mix, out_w=pending.out_w, bias=pending.bias,
+                        identity=pending.identity, **kw)
         return buf
 
     def forward(self, X, pending, ctx, cache):
@@ -366,9 +370,14 @@ class HyperBlock:
         pending = HyperPending(y, self.hc[names[0]][2], self.hc[names[0]][1], self.spec.mixer_norm.eps,
                                bias=self.mixer.out_bias if getattr(self.mixer, "defer_bias", False) else None)
         if self.ffn is not None:
+            keeps = getattr(self.ffn, "n_identity", 0)       # what it read is read again behind it: not the next norm's buffer
+            if keeps:
+                buf = ctx.ws.buf("normed_kept", n, H, self.dtype)
             x = self._between(X, pending, names[1], self.ffn_norm, buf)
             y = self.ffn.forward(x, ctx)
-            pending = HyperPending(y, self.hc[names[1]][2], self.hc[names[1]][1], self.spec.ffn_norm.eps)
+            pending = HyperPending(y, self.hc[names[1]][2], self.hc[names[1]][1], self.spec.ffn_norm.eps,
+                                   bias=self.ffn.out_bias if getattr(self.ffn, "defer_bias", False) else None,
+                                   identity=self.ffn.identity if keeps else None)
         return pending
 
 

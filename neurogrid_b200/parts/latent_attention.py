@@ -32,6 +32,7 @@ class LatentAttention:
     the core's dot product over the whole row is the sum of the two scores; the head's weighted rows carry r
     coordinates that nothing reads.  With a gate per element (``spec.gate`` "element") W_uv cannot be folded into the
     output projection: a kernel expands each head's weighted latent by W_uv,h and applies the gate, then W_o follows.
+    With no gate (``spec.gate`` "none") the expansion to values is folded into the output projection, as for a gate per head.
     ``owns_cache`` False builds a layer that reads another latent layer's pages: it has no W_dkv and no norm of c."""
 
     graph_safe = True      # launches depend on device data and on launch-time constants only
@@ -45,7 +46,7 @@ class LatentAttention:
         if not owns_cache and not self.rope and not self.by_element:
             raise ValueError("a latent attention layer of this form keeps its own cache")
         self.rank_p = -(-(spec.kv_rank + self.rope) // 16) * 16
-        self.n_gate = spec.n_heads * spec.value_dim if self.by_element else spec.n_heads
+        self.n_gate = spec.n_heads * spec.value_dim if self.by_element else 0 if spec.gate == "none" else spec.n_heads
         self.position = registry.build("position", spec.position, device=device) if self.rope else None
         self.w_down = self.w_q = self.w_out = self.w_uv = self.dq_norm = self.dkv_norm = None
 
@@ -55,8 +56,9 @@ class LatentAttention:
              n["uq"]: TensorDecl((s.n_heads * (s.key_dim + self.rope), s.q_rank)),
              n["uk"]: TensorDecl((s.n_heads * s.key_dim, s.kv_rank)),
              n["uv"]: TensorDecl((s.n_heads * s.value_dim, s.kv_rank)),
-             n["gate"]: TensorDecl((self.n_gate, s.hidden)),
              n["o"]: TensorDecl((s.hidden, s.n_heads * s.value_dim))}
+        if self.n_gate:
+            d[n["gate"]] = TensorDecl((self.n_gate, s.hidden))
         if self.owns_cache:
             d[n["dkv"]] = TensorDecl((s.kv_rank + self.rope, s.hidden))
             d[n["dkv_norm"]] = TensorDecl((s.kv_rank,), "norm")
@@ -67,7 +69,7 @@ class LatentAttention:
         kw = dict(device=self.device, dtype=self.dtype)
         f32 = dict(device=self.device, dtype=torch.float32)
         H, rp = s.n_heads, self.rank_p
-        self.w_down = torch.cat([t[n[p]].to(**kw) for p in (("dq", "dkv", "gate") if self.owns_cache else ("dq", "gate"))]).contiguous()
+        self.w_down = torch.cat([t[n[p]].to(**kw) for p in ("dq",) + (("dkv",) if self.owns_cache else ()) + (("gate",) if self.n_gate else ())]).contiguous()
         self.dq_norm = t[n["dq_norm"]].to(**f32).contiguous()
         self.dkv_norm = t[n["dkv_norm"]].to(**f32).contiguous() if self.owns_cache else None
         uq = t[n["uq"]].double().view(H, s.key_dim + self.rope, s.q_rank)
@@ -94,8 +96,6 @@ class LatentAttention:
         the encoding's rotated coordinates get the frequency zero (they pass unchanged)."""
         if getattr(self, "_pa", None) is None:
             pa = PositionArgs.of(self.position.kernel_args())
-            if pa.magnitude != 1.0:
-                raise NotImplementedError("the rotated part takes rotations that keep lengths")
             if pa.pos_scale != 1.0 or (pa.half_pairing and pa.inv_freq is not None and pa.inv_freq.numel() != self.rope // 2):
                 raise NotImplementedError("the rotated part takes unscaled positions, and pairs (i, i + half) only whole")
             f = torch.zeros(self.rope // 2, dtype=torch.float32, device=self.device)
@@ -128,16 +128,16 @@ class LatentAttention:
         down = ctx.ws.buf("lat_down", n, w_down.shape[0], self.dtype)
         ops.linear(x, w_down, None, down)
         cq = ctx.ws.buf("lat_cq", n, s.q_rank, self.dtype)
-        gate = ctx.ws.buf("lat_gate", n, self.n_gate, torch.float32)
+        gate = ctx.ws.buf("lat_gate", n, self.n_gate, torch.float32) if self.n_gate else None
         pa = self._position_args() if self.rope else None
         ops.latent_prep(down, self.dq_norm, self.dkv_norm if writes else None, cq, cache.k_pages if writes else None, gate,
                         cache.table, ctx.positions, ctx.row_entry, self.n_gate, s.eps, ctx.status,
                         rot=self.rope if writes else 0, inv_freq=pa.inv_freq if pa else None,
-                        half_pairing=bool(pa and pa.half_pairing))
+                        half_pairing=bool(pa and pa.half_pairing), rot_mag=pa.magnitude if pa else 1.0)
         q = ctx.ws.buf("lat_q", n, H * rp, self.dtype)
         ops.linear(cq, self.w_q, None, q)
         if self.rope:
-            ops.latent_rope_q(q, ctx.positions, ctx.row_entry, pa.inv_freq, H, s.kv_rank, pa.half_pairing)
+            ops.latent_rope_q(q, ctx.positions, ctx.row_entry, pa.inv_freq, H, s.kv_rank, pa.half_pairing, rot_mag=pa.magnitude)
         o = ctx.ws.buf("lat_o", n, H * rp, self.dtype)
         head_gate = None if self.by_element else gate
         if n > self.SPLIT_MAX_ROWS and ops.latent_core_mma_takes(H, rp, self.dtype):

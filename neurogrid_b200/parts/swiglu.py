@@ -18,21 +18,34 @@ class SwiGLU:
 
     def __init__(self, spec, *, dtype, device):
         self.spec, self.dtype, self.device = spec, dtype, device
-        self.w_gate_up = self.w_down = None
+        self.w_gate_up = self.w_down = self.b_gate_up = self.b_down = None
+        self.out_bias = None          # the down projection's bias in float32, for a block that adds it itself
+        self.defer_bias = False       # set by such a block
 
     def _name(self, role):
         return self.spec.names[role] + getattr(self.spec, "weight_suffix", ".weight")
 
+    def _bias_name(self, role):
+        return self.spec.names[role] + self.spec.bias_suffix
+
     def tensors(self):
         s = self.spec
-        return {self._name("gate"): TensorDecl((s.intermediate, s.hidden)),
-                self._name("up"): TensorDecl((s.intermediate, s.hidden)),
-                self._name("down"): TensorDecl((s.hidden, s.intermediate))}
+        d = {self._name("gate"): TensorDecl((s.intermediate, s.hidden)),
+             self._name("up"): TensorDecl((s.intermediate, s.hidden)),
+             self._name("down"): TensorDecl((s.hidden, s.intermediate))}
+        if getattr(s, "bias", False):
+            for role, rows in (("gate", s.intermediate), ("up", s.intermediate), ("down", s.hidden)):
+                d[self._bias_name(role)] = TensorDecl((rows,), "bias")
+        return d
 
     def bind(self, t):
         kw = dict(device=self.device, dtype=self.dtype)
         self.w_gate_up = torch.cat([t[self._name("gate")].to(**kw), t[self._name("up")].to(**kw)]).contiguous()
         self.w_down = t[self._name("down")].to(**kw).contiguous()
+        if getattr(self.spec, "bias", False):
+            self.b_gate_up = torch.cat([t[self._bias_name(r)].to(**kw) for r in ("gate", "up")]).contiguous()
+            self.b_down = t[self._bias_name("down")].to(**kw).contiguous()
+            self.out_bias = t[self._bias_name("down")].to(device=self.device, dtype=torch.float32).contiguous()
 
     def kernels(self):
         return [("gemm_sm100" if self.dtype == torch.bfloat16 else "gemm_f32", None), ("elementwise", None)]
@@ -41,7 +54,7 @@ class SwiGLU:
         s = self.spec
         act = ctx.ws.buf("ffn_act", x.shape[0], s.intermediate, self.dtype)
         self.gated(x, ctx, act)
-        return ops.linear_to_residual(act, self.w_down, None, ctx.ws, "ffn_out", residual=ctx.residual)
+        return ops.linear_to_residual(act, self.w_down, None if self.defer_bias else self.b_down, ctx.ws, "ffn_out", residual=ctx.residual)
 
     # For a block arrangement that ends mixer and feed-forward with ONE product: the gated activations go into a
     # block of columns of the caller's buffer, and the caller multiplies by ``out_weight()``.
@@ -49,7 +62,7 @@ class SwiGLU:
         return self.spec.intermediate
 
     def out_weight(self):
-        return self.w_down, None
+        return self.w_down, self.b_down
 
     def drop_out_weight(self):
         """The caller keeps a stacked copy of the output matrix and will not call ``forward``."""
@@ -62,8 +75,8 @@ class SwiGLU:
         if kw["activation"] == "clamped_glu":
             kw.update(limit=s.limit, alpha=s.glu_alpha)
         if ops.gemm_sm100_ok(x, self.w_gate_up):
-            ops.gemm_swiglu_sm100(x, self.w_gate_up, act, **kw)    # the gate rides in the epilogue
+            ops.gemm_swiglu_sm100(x, self.w_gate_up, act, bias=self.b_gate_up, **kw)    # the gate rides in the epilogue
         else:
             gu = ctx.ws.buf("ffn_gate_up", x.shape[0], 2 * s.intermediate, self.dtype)
-            ops.linear(x, self.w_gate_up, None, gu)
+            ops.linear(x, self.w_gate_up, self.b_gate_up, gu)
             ops.swiglu(gu, act, **kw)

@@ -83,13 +83,19 @@ def add_layernorm(h, delta, weight, out, eps, rows=None, post=None):
 
 def qkv_prep(qkv, q_out, q_weight, k_weight, inv_freq, k_pages, v_pages, table, positions, row_entry, n_q, n_k, n_v,
              dim, vdim, eps, status, *, whole=False, q_temp_coef=0.0, q_temp_every=1, half_pairing=False, unit_norm=False,
-             v_is_k=False, rot_mag=1.0):
+             v_is_k=False, rot_mag=1.0, v_norm=False, v_first=None, v_lambda=None):
     n = qkv.shape[0]
     x = qkv.to(D)
     q = x[:, : n_q * dim].reshape(n, n_q, dim)
     k = x[:, n_q * dim:(n_q + n_k) * dim].reshape(n, n_k, dim)
     v_at = (n_q if v_is_k else n_q + n_k) * dim                   # columns behind v are the caller's
     v = x[:, v_at:v_at + n_v * vdim].reshape(n, n_v, vdim)
+    if v_norm:
+        v = v * torch.rsqrt((v * v).mean(-1, keepdim=True) + eps)
+    if v_lambda is not None:
+        v = (1.0 - v_lambda) * v + v_lambda * v_first.to(D).reshape(v.shape)
+    elif v_first is not None:
+        v_first.copy_(v.reshape(n, -1).to(v_first.dtype))
 
     def norm(t, w):
         if w is None and unit_norm:
@@ -141,7 +147,7 @@ def qkv_prep(qkv, q_out, q_weight, k_weight, inv_freq, k_pages, v_pages, table, 
 
 def mapped_attention(q, k_pages, v_pages, table, positions, row_entry, out, n_heads, n_maps, window, keep_first, scale,
                      softcap, lam, head_norm, post_scale, eps, n_splits=1, partial=None, slopes=None, sinks=None, chunk=0,
-                     out_scale=1.0):
+                     out_scale=1.0, sigmoid=False, score_bias=None, gate=None):
     n = q.shape[0]
     P, n_k, ps, dim = k_pages.shape
     n_g, vdim = v_pages.shape[1], v_pages.shape[3]
@@ -170,7 +176,9 @@ def mapped_attention(q, k_pages, v_pages, table, positions, row_entry, out, n_he
                     s = softcap * torch.tanh(s / softcap)
                 if slopes is not None:
                     s = s - slopes[h].to(D) * (pos - kp).to(D)
-                if sinks is not None:                              # one more term of the denominator, without a value
+                if sigmoid:
+                    w = torch.sigmoid(s + (score_bias[h].to(D) if score_bias is not None else 0.0))
+                elif sinks is not None:                            # one more term of the denominator, without a value
                     w = torch.softmax(torch.cat([s, sinks[h].to(D).reshape(1)]), 0)[:-1]
                 else:
                     w = torch.softmax(s, 0)
@@ -178,6 +186,8 @@ def mapped_attention(q, k_pages, v_pages, table, positions, row_entry, out, n_he
             y = a[0] if n_maps == 1 else a[0] - lam * a[1]
             if head_norm:
                 y = y * torch.rsqrt((y * y).mean() + eps) * post_scale
+            if gate is not None:
+                y = y * torch.sigmoid(gate[r, h].to(D))
             o[h] = y * out_scale
         out[r] = o.reshape(-1).to(out.dtype)
 
@@ -261,7 +271,7 @@ def softcap_(x, cap):
 
 
 def moe_router_sigmoid(x, w_router, correction, w_shared_gate, weights, top_k, n_groups=1, keep_groups=1, *,
-                       softmax_scores=False, group_max=False, route_scale=1.0):
+                       softmax_scores=False, group_max=False, route_scale=1.0, n_identity=0):
     n, E = x.shape[0], w_router.shape[0]
     logits = x.to(D) @ w_router.to(D).T
     s = torch.softmax(logits, -1) if softmax_scores else torch.sigmoid(logits)
@@ -281,9 +291,9 @@ def moe_router_sigmoid(x, w_router, correction, w_shared_gate, weights, top_k, n
         chosen = sorted(range(E), key=lambda e: (-float(c[e]), e))[:top_k]
         total = sum(float(s[r, e]) for e in chosen) + 1e-20
         for e in chosen:
-            weights[r, e] = float(s[r, e]) / total * route_scale
+            weights[r, e if e < E - n_identity else -1] += float(s[r, e]) / total * route_scale
     if w_shared_gate is not None:
-        weights[:, E] = torch.sigmoid(x.to(D) @ w_shared_gate.to(D)).to(weights.dtype)
+        weights[:, E - n_identity] = torch.sigmoid(x.to(D) @ w_shared_gate.to(D)).to(weights.dtype)
 
 
 def moe_clamped_glu_scaled(gate_up, weights, out, n_experts, expert_ff, limit, shared_limit, alpha, shared_gated):
@@ -449,7 +459,7 @@ def gate_mul(y, gate, activation="sigmoid", scale=1.0):
 
 
 def hc_step(streams, n_streams, *, x0=None, delta=None, mix=None, out_w=None, in_w=None, norm_w=None, out=None, sum_out=None,
-            eps=0.0, act_dtype=None, bias=None):
+            eps=0.0, act_dtype=None, bias=None, identity=None):
     n, S = streams.shape[0], n_streams
     H = streams.shape[1] // S
     X = x0.to(D)[:, None, :].expand(n, S, H).clone() if x0 is not None else streams.to(D).reshape(n, S, H)
@@ -457,6 +467,8 @@ def hc_step(streams, n_streams, *, x0=None, delta=None, mix=None, out_w=None, in
         y = (delta.sum(0) if delta.dim() == 3 else delta).to(D)
         if bias is not None:
             y = y + bias.to(D)
+        if identity is not None:
+            y = y + identity[1].to(D)[:, None] * identity[0].to(D)
         X = torch.einsum("st,nsh->nth", mix.to(D).reshape(S, S), X) + out_w.to(D)[None, :, None] * y[:, None, :]
     if x0 is not None or delta is not None:
         streams.copy_(X.reshape(n, S * H).to(streams.dtype))
@@ -467,9 +479,13 @@ def hc_step(streams, n_streams, *, x0=None, delta=None, mix=None, out_w=None, in
         sum_out.copy_(X.sum(1).to(sum_out.dtype))
 
 
-def moe_swiglu_scaled(gate_up, weights, out, expert_ff, shared_gated=False):
+def moe_identity_add(y, x, w):
+    y.copy_((y.to(D) + w.to(D)[:, None] * x.to(D)).to(y.dtype))
+
+
+def moe_swiglu_scaled(gate_up, weights, out, expert_ff, shared_gated=False, n_experts=None):
     n, I = out.shape
-    E = weights.shape[1] - int(bool(shared_gated))
+    E = weights.shape[1] - int(bool(shared_gated)) if n_experts is None else n_experts
     g, u = gate_up[:, :I].to(D), gate_up[:, I:].to(D)
     w = weights[:, :E].to(D).repeat_interleave(expert_ff, dim=1)
     tail = weights[:, E:E + 1].to(D) if shared_gated else torch.ones(n, 1, dtype=D)
@@ -558,18 +574,19 @@ def mlstm(x, gates, gate_bias, cap, norm_w, state, nm_state, o_raw, out, cu_q, c
 
 
 def latent_prep(x, wq, wkv, cq_out, pages, gate_out, table, positions, row_entry, n_heads, eps, status, *, rot=0,
-                inv_freq=None, half_pairing=False):
+                inv_freq=None, half_pairing=False, rot_mag=1.0):
     n, rq = cq_out.shape
     rkv = wkv.numel() if wkv is not None else 0
     xd = x.to(D)
     a = xd[:, :rq]
     cq_out.copy_((a * torch.rsqrt((a * a).mean(-1, keepdim=True) + eps) * wq.to(D)).to(cq_out.dtype))
-    gate_out.copy_(torch.sigmoid(xd[:, rq + rkv + rot:]).to(gate_out.dtype))
+    if gate_out is not None:
+        gate_out.copy_(torch.sigmoid(xd[:, rq + rkv + rot:]).to(gate_out.dtype))
     if not rkv:
         return
     c = xd[:, rq:rq + rkv]
     c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * wkv.to(D)
-    kr = _rotate_tail(xd[:, rq + rkv:rq + rkv + rot], positions, inv_freq, half_pairing) if rot else xd[:, :0]
+    kr = _rotate_tail(xd[:, rq + rkv:rq + rkv + rot], positions, inv_freq, half_pairing, rot_mag) if rot else xd[:, :0]
     ps, rp = pages.shape[2], pages.shape[3]
     for r in range(n):
         e = int(row_entry[r])
@@ -582,10 +599,10 @@ def latent_prep(x, wq, wkv, cq_out, pages, gate_out, table, positions, row_entry
         pages[page, 0, pos % ps] = rowv.to(pages.dtype)
 
 
-def _rotate_tail(t, positions, inv_freq, half_pairing):
+def _rotate_tail(t, positions, inv_freq, half_pairing, rot_mag=1.0):
     r = t.shape[-1]
     ang = (positions.to(torch.float32)[:, None] * inv_freq[None, :]).to(D)
-    c, s = torch.cos(ang), torch.sin(ang)
+    c, s = rot_mag * torch.cos(ang), rot_mag * torch.sin(ang)
     o = t.clone()
     if half_pairing:
         a, b = t[..., :r // 2], t[..., r // 2:]
@@ -596,13 +613,13 @@ def _rotate_tail(t, positions, inv_freq, half_pairing):
     return o
 
 
-def latent_rope_q(q, positions, row_entry, inv_freq, n_heads, offset, half_pairing=False):
+def latent_rope_q(q, positions, row_entry, inv_freq, n_heads, offset, half_pairing=False, rot_mag=1.0):
     n = q.shape[0]
     rot = 2 * inv_freq.numel()
     qv = q.view(n, n_heads, -1)
     for h in range(n_heads):
         qv[:, h, offset:offset + rot] = _rotate_tail(qv[:, h, offset:offset + rot].to(D), positions, inv_freq,
-                                                     half_pairing).to(q.dtype)
+                                                     half_pairing, rot_mag).to(q.dtype)
 
 
 def latent_core(q, pages, table, positions, row_entry, gate, out, n_heads, window, scale, n_splits=1, partial=None):
@@ -634,7 +651,7 @@ def head_up_gate(o, w, gate, out):
     out.copy_(y.to(out.dtype))
 
 
-_NAMES = ["embed_norm", "lightning", "mlstm", "scale_", "gate_mul", "hc_step", "moe_swiglu_scaled", "gated_linear", "latent_prep", "latent_rope_q", "latent_core",
+_NAMES = ["embed_norm", "lightning", "mlstm", "scale_", "gate_mul", "hc_step", "moe_swiglu_scaled", "moe_identity_add", "gated_linear", "latent_prep", "latent_rope_q", "latent_core",
           "head_up_gate", "gather_tokens", "embed", "add_rmsnorm", "residual_add", "swiglu", "gemm_f32", "linear", "shortconv", "rope_cache",
           "attention_generic", "sample", "add_layernorm", "qkv_prep", "mapped_attention", "gated_delta", "pair_embed",
           "pair_norm_mean", "relu_squared_", "softcap_", "moe_router_sigmoid", "moe_clamped_glu_scaled"]
