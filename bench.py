@@ -2,7 +2,7 @@
 """Decode and prefill throughput of the engine at the LFM2-1.2B shape, random weights, one B200.
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--layers N] [--impl ours|reference]
-                    [--shape 1.2b|700m|350m] [--prompt-len N] [--workload mixed350m|long700m|metanex|rofulorn|fuzelorn|dodilix|matepel]
+                    [--shape 1.2b|700m|350m] [--prompt-len N] [--workload mixed350m|long700m|metanex|rofulorn|fuzelorn|dodilix|matepel|pepulix]
 
 A "step" is one decode step of the batch.  The default run has the layer sizes of the
 LFM2-1.2B configuration, a batch of 8 and requests that hold 2,048-token prompts and grow
@@ -1478,6 +1478,179 @@ def matepel_kernel_times(eng, l2, pk):
     return out
 
 
+# ---------------------------------------------------------------------------------------------- --workload pepulix
+def pepulix_config(width, layers):
+    """A Pepulix configuration with layers of a real model's sizes: four copies of the stream; every other layer an mLSTM
+    (heads of 128 x 128) with a dense feed-forward four widths wide, between them in turn a sigmoid attention (heads of
+    128 with half of each head rotated, four query heads to a key/value head, values mixed with the first such layer's)
+    and a latent attention (heads of 128 + 64 rotated coordinates with rescaled frequencies, a latent of 192 beside the 64
+    shared rotated ones, queries through a latent of width/2), both with 16 routed experts of width/4 and four identity
+    experts, top 4."""
+    heads = width // 128
+    attention = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+                 "rot": {"base": 10000.0, "dims": 64}}
+    latent = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "q_rank": width // 2, "kv_rank": 192, "scale": 192 ** -0.5,
+              "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 2.0}}}
+    mlstm = {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 12.0}
+    moe = {"kind": "moe", "router": {"experts": 16, "identity": 4, "top": 4}, "expert": {"ff": width // 4}}
+    dense = {"kind": "dense", "ff": 4 * width}
+    kinds = [("mlstm", mlstm, dense), ("attention", attention, moe), ("mlstm", mlstm, dense), ("latent_attention", latent, moe)]
+    out = [{"type": t, "mixer": m, "mlp": f} for t, m, f in (kinds[i % 4] for i in range(layers))]
+    return {"architecture": "Pepulix", "vocab": 65536, "width": width, "streams": 4, "norm": {"eps": 1e-5}, "logit_softcap": 40.0,
+            "layers": out}
+
+
+def run_pepulix(args):
+    """Prefill and decode throughput of the Pepulix design at layer sizes of a real model, beside the two existing models
+    it is closest to at equal width and depth: Dodilix (copies of the stream, latent attention, routed experts) and
+    Matepel (copies of the stream, causal attention with float32 weights, an mLSTM), and the designs' own kernels one by
+    one.  One JSON line.  Random weights, synthetic token ids; CUDA events; the L2 is flushed between timed steps."""
+    import torch
+    pk = peaks()
+    l2 = torch.zeros(256 << 20, dtype=torch.uint8, device="cuda:0")
+    clocks = ClockSampler(0)
+    clocks.start()
+    results = []
+    kernels = {"pepulix": pepulix_kernel_times, "dodilix": dodilix_kernel_times, "matepel": matepel_kernel_times}
+    for width, layers in ((1024, 16), (2048, 16)):
+        row = {"width": width, "layers": layers}
+        for arm, cfg in {"pepulix": pepulix_config(width, layers), "dodilix": dodilix_config(width, layers),
+                         "matepel": matepel_config(width, layers)}.items():
+            eng = design_arm(arm, cfg, row, args, l2)
+            if not args.no_kernels:
+                row[arm + "_kernels"] = kernels[arm](eng, l2, pk)
+            del eng
+            torch.cuda.empty_cache()
+        results.append(row)
+    time.sleep(0.06)
+    clocks.stop()
+    print(json.dumps({"workload": "pepulix", "what": "Pepulix beside Dodilix and Matepel at equal width and depth: prefill of "
+                      "2,048 tokens, decode at batch 8 and 1 after 2,048 tokens; each design's own kernels alone",
+                      "results": results, "dtype": "bf16", "data": "synthetic token ids, random-init weights", "peaks": pk,
+                      "clocks": clocks.summary(), "impl": "ours"}))
+
+
+def pepulix_kernel_times(eng, l2, pk):
+    """The design's own kernels alone, through the parts' own launch plans (CUDA events around the launches, L2 flushed
+    before, median of 7), for a 2,048-token portion and for 8 single tokens after 2,048: microseconds, the bytes each
+    must move with the fraction of the measured copy bandwidth, and for the recurrence and the attention cores the
+    multiply-adds they must do as TFLOP/s."""
+    import torch
+    from neurogrid_b200.csrc import ops
+    from neurogrid_b200.parts import PagedView, StepContext
+    from neurogrid_b200.parts.base import Workspace
+    model, dev = eng.model, eng.device
+    D, S = model.spec.hidden, model.spec.streams
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+    g = torch.Generator(device=dev).manual_seed(3)
+    rnd = lambda *s: torch.randn(*s, generator=g, device=dev).to(torch.bfloat16)
+    bf = lambda *s: torch.empty(*s, dtype=torch.bfloat16, device=dev)
+
+    def timed(fn):
+        fn()
+        torch.cuda.synchronize()
+        ts = []
+        for _ in range(9):
+            flush_l2(l2)
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            fn()
+            b.record()
+            torch.cuda.synchronize()
+            ts.append(a.elapsed_time(b) * 1e3)
+        return median(ts[2:])
+
+    out = {"unit": "us"}
+    bw = pk["hbm_gbs"] * 1e9
+
+    def mem(name, us, nbytes, flops=0, tensor=False):
+        out[name] = {"us": round(us, 2), "bytes": int(nbytes), "of_copy_bandwidth": round(nbytes / (us * 1e-6) / bw, 3)}
+        if flops:
+            out[name]["flops"] = int(flops)
+            out[name]["tflops"] = round(flops / (us * 1e-6) / 1e12, 2)
+        if tensor:
+            out[name]["of_tensor_peak"] = round(flops / (us * 1e-6) / 1e12 / pk["bf16_tflops"], 4)
+
+    by_kind = lambda name: [b for b in model.blocks if type(b.mixer).__name__ == name]
+    att_block, lat_block, rec_block = by_kind("MappedAttention")[1], by_kind("LatentAttention")[0], by_kind("MLSTM")[0]
+    att, lat, rec, f = att_block.mixer, lat_block.mixer, rec_block.mixer, lat_block.ffn
+    sa, sl, sr, fs = att.spec, lat.spec, rec.spec, f.spec
+    need = att.cache_need()
+    ps, n_pages = 16, 8 * 4096 // 16
+    kp, vp = rnd(n_pages, need.n_kv_heads, ps, need.head_dim), rnd(n_pages, need.value_shape()[0], ps, need.value_shape()[1])
+    lp = rnd(n_pages, 1, ps, lat.rank_p)
+    for rows, entries in ((PREFILL_TOKENS, 1), (8, 8)):
+        tag = "prefill2048" if entries == 1 else "decode8"
+        q_len = rows // entries
+        before = 0 if entries == 1 else 2048
+        table = torch.arange(entries * 256, dtype=torch.int32, device=dev).view(entries, 256)
+        ctx = StepContext(n_rows=rows, n_entries=entries, max_q=q_len, tokens=i32([0] * rows),
+                          positions=i32([before + t for e in range(entries) for t in range(q_len)]),
+                          row_entry=i32([e for e in range(entries) for _ in range(q_len)]),
+                          cu_q=i32([q_len * e for e in range(entries + 1)]), ctx_before=i32([before] * entries),
+                          slots=i32(list(range(entries))), status=torch.zeros(1, dtype=torch.int32, device=dev),
+                          ws=Workspace(4096, dev), dtype=torch.bfloat16, q_lens=[q_len] * entries,
+                          ctx_lens=[before] * entries, slot_ids=list(range(entries)))
+        pairs = sum(t + 1 for t in range(rows)) if entries == 1 else rows * (before + 1)
+        # between two sublayers: the copies' update with what a feed-forward hands over (a bias; identity experts)
+        X, y, z = torch.randn(rows, S * D, generator=g, device=dev), rnd(rows, D), rnd(rows, D)
+        wts = torch.rand(rows, fs.n_experts + 1, generator=g, device=dev)
+        w_in, w_out, mix = rec_block.hc["hc1"]
+        normed = bf(rows, D)
+        kw = dict(delta=y, mix=mix, out_w=w_out, in_w=w_in, norm_w=rec_block.mixer_norm.weight, out=normed, eps=1e-5)
+        mem(f"{tag}_stream_copies", timed(lambda: ops.hc_step(X, S, bias=rec_block.ffn.out_bias, **kw)), rows * D * (2 * 4 * S + 2 + 2))
+        mem(f"{tag}_stream_copies_identity", timed(lambda: ops.hc_step(X, S, identity=(z, wts[:, fs.n_experts]), **kw)),
+            rows * D * (2 * 4 * S + 2 + 2 + 2))
+        # sigmoid attention: rotation, norms, mixed values, page write; the core with the gate per head
+        d, dv, H, G = sa.key_dim, sa.value_dim, sa.n_heads, sa.n_kv_heads
+        qkv, qb, o = rnd(rows, att.w_qkv.shape[0]), bf(rows, H * d), bf(rows, H * dv)
+        first = torch.randn(rows, G * dv, generator=g, device=dev)
+        pa = att.position.kernel_args()
+        view = PagedView(kp, vp, table)
+        gate = qkv[:, (H + G) * d + G * dv:][:, :H]
+        mem(f"{tag}_attention_prep", timed(lambda: ops.qkv_prep(
+            qkv, qb, None, None, pa.inv_freq, kp, vp, table, ctx.positions, ctx.row_entry, H, G, G, d, dv, sa.eps, ctx.status,
+            half_pairing=True, unit_norm=True, v_norm=True, v_first=first, v_lambda=0.3)),
+            rows * (2 * (H + G) * d * 2 + 2 * G * dv * 2 + G * dv * 4))
+        mem(f"{tag}_attention_core", timed(lambda: att.attend(qb, view, ctx, o, None, 1.0, gate)),
+            entries * (before + q_len) * need.elements_per_token() * 2 + 2 * rows * H * d * 2, 2 * pairs * H * (d + dv), True)
+        # the recurrence with its gates, norm and output gate
+        nH, dk, dvr = sr.n_heads, sr.key_dim, sr.value_dim
+        p, gates = rnd(rows, rec.w_in.shape[0]), torch.randn(rows, 2 * nH, generator=g, device=dev)
+        state = torch.zeros(8, nH, dk, dvr, device=dev)
+        nm = torch.zeros(8, nH, ops.decayed_linear_slices(dvr), dk + 1, device=dev)
+        raw, og, scratch = torch.empty(rows, nH * dvr, device=dev), bf(rows, nH * dvr), rec._chunk_scratch(ctx, rows)
+        mem(f"{tag}_mlstm", timed(lambda: ops.mlstm(
+            p, gates, rec.b_gates, sr.gate_cap, rec.norm, state, nm, raw, og, ctx.cu_q, ctx.ctx_before, ctx.slots, ctx.row_entry,
+            entries, nH, dk, dvr, sr.eps, 1.0, scratch=scratch, max_q=q_len)),
+            (p.numel() + og.numel()) * 2 + 2 * entries * state[0].numel() * 4, 4 * rows * nH * dk * dvr)
+        # latent attention: the row kernel, the rotation of q, the core, the product that expands the values and projects
+        Hl, rp = sl.n_heads, lat.rank_p
+        down, cq, la = rnd(rows, lat.w_down.shape[0]), bf(rows, sl.q_rank), lat._position_args()
+        mem(f"{tag}_latent_prep", timed(lambda: ops.latent_prep(
+            down, lat.dq_norm, lat.dkv_norm, cq, lp, None, table, ctx.positions, ctx.row_entry, 0, sl.eps, ctx.status, rot=lat.rope,
+            inv_freq=la.inv_freq, rot_mag=la.magnitude)), down.numel() * 2 + cq.numel() * 2 + rows * rp * 2)
+        ql, ol = rnd(rows, Hl * rp), bf(rows, Hl * rp)
+        mem(f"{tag}_latent_rope_q", timed(lambda: ops.latent_rope_q(ql, ctx.positions, ctx.row_entry, la.inv_freq, Hl, sl.kv_rank,
+                                                                    rot_mag=la.magnitude)), 2 * rows * Hl * lat.rope * 2)
+        mem(f"{tag}_latent_core", timed(lambda: lat.attend(ql, PagedView(lp, None, table), ctx, ol)),
+            entries * (before + q_len) * rp * 2 + 2 * rows * Hl * rp * 2, 4 * pairs * Hl * rp, True)
+        mem(f"{tag}_latent_out_product", timed(lambda: ops.linear_to_residual(ol, lat.w_out, None, ctx.ws, "out")),
+            ol.numel() * 2 + lat.w_out.numel() * 2 + rows * D * 2, 2 * rows * lat.w_out.numel(), True)
+        # router and the activation with the routing weights; the dense feed-forward's gate
+        mem(f"{tag}_moe_router", timed(lambda: ops.moe_router_sigmoid(
+            z, f.w_router, f.correction, None, wts, fs.top_k, softmax_scores=True, n_identity=fs.identity)),
+            rows * D * 2 + f.w_router.numel() * 4 + wts.numel() * 4)
+        gu, act = rnd(rows, 2 * f.width), bf(rows, f.width)
+        mem(f"{tag}_moe_activation", timed(lambda: ops.moe_swiglu_scaled(gu, wts, act, fs.expert_ff, n_experts=fs.n_experts)),
+            3 * rows * f.width * 2)
+        if entries == 1:
+            I = rec_block.ffn.spec.intermediate
+            gu, act = rnd(rows, 2 * I), bf(rows, I)
+            mem(f"{tag}_swiglu", timed(lambda: ops.swiglu(gu, act)), 3 * rows * I * 2)
+    return out
+
+
 def run_reference(args):
     """The reference's own library through its stock entry points; same metric, same line."""
     shape_name = SHAPE_NAMES[args.shape]
@@ -1540,7 +1713,8 @@ def main():
     ap.add_argument("--prompt-len", type=int, default=0,
                     help="tokens each request holds before decoding (default 2,048; the context is twice this)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
-    ap.add_argument("--workload", default="", choices=["", "mixed350m", "long700m", "metanex", "rofulorn", "fuzelorn", "dodilix", "matepel"],
+    ap.add_argument("--workload", default="", choices=["", "mixed350m", "long700m", "metanex", "rofulorn", "fuzelorn", "dodilix", "matepel",
+                                                          "pepulix"],
                     help="run another workload of the benchmark set through Engine.generate instead; metanex / rofulorn: "
                          "that design beside LFM2 at equal width and depth, prefill and decode, and its kernels alone")
     ap.add_argument("--repeat", type=int, default=2, help="--workload: runs (the first also warms up and captures graphs)")
@@ -1559,6 +1733,9 @@ def main():
         args.warmup = 3
     if args.workload == "metanex":
         run_metanex(args)
+        return 0
+    if args.workload == "pepulix":
+        run_pepulix(args)
         return 0
     if args.workload == "matepel":
         run_matepel(args)

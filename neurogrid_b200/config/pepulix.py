@@ -133,9 +133,9 @@ class PepulixConfig:
             if t == "attention":
                 _check_attention(m, mp)
                 if m.get("v_mix"):
-                    values = m["kv_heads"] * m["vdim"]
+                    values = (m["kv_heads"], m["vdim"])
                     if mixing is not None and values != mixing[1]:
-                        raise ConfigError(f"{mp}v_mix: kv_heads * vdim = {values} differs from layers[{mixing[0]}]'s {mixing[1]}")
+                        raise ConfigError(f"{mp}v_mix: (kv_heads, vdim) = {values} differs from layers[{mixing[0]}]'s {mixing[1]}")
                     mixing = mixing or (i, values)
             elif t == "latent_attention":
                 _check_latent(m, mp)

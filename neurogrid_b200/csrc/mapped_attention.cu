@@ -33,7 +33,8 @@
 #define MA_MAX_PAIRS 8    // pairs of a head per lane in the prep kernel: d <= 512
 
 // ------------------------------------------------------------------------------------------ prep
-template <typename T>
+// OWN_V: value heads are normed or mixed (a form of its own: the others' values are copied as they are)
+template <typename T, bool OWN_V>
 __global__ void __launch_bounds__(MA_THREADS)
 qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* __restrict__ qw,
                 const float* __restrict__ kw, const float* __restrict__ inv_freq, int rot_dims,
@@ -148,7 +149,7 @@ qkv_prep_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, const float* _
     }
     if (page_ok) {
         const T* vs = in + (size_t)(v_is_k ? nQ : nQ + nK) * d;      // v_is_k: the values are the keys as projected
-        if (v_norm || v_mode) {                          // a warp per value head, float32 until the store
+        if (OWN_V) {                                     // a warp per value head, float32 until the store
             v_first = ng_after_wait(v_first);
             for (int hv = blockIdx.y * MA_WARPS + warp; hv < nV; hv += MA_WARPS * gridDim.y) {
                 float v[2 * MA_DVU], ss = 0.f;
@@ -198,15 +199,19 @@ NG_EXPORT int ng_qkv_prep(const void* qkv, void* q_out, const float* qw, const f
     const size_t smem = (size_t)rot_dims * sizeof(float);
     const int head_blocks = n_rows >= 256 ? 1 : min(64, (nQ + nK + MA_WARPS - 1) / MA_WARPS);
     const dim3 grid(n_rows, head_blocks);
-    if (act_bf16)
-        NG_LAUNCH((qkv_prep_kernel<__nv_bfloat16>), grid, MA_THREADS, smem, stream, (const __nv_bfloat16*)qkv,
-                  (__nv_bfloat16*)q_out, qw, kw, inv_freq, rot_dims, (__nv_bfloat16*)k_pages, (__nv_bfloat16*)v_pages, table,
-                  table_stride, positions, row_entry, nQ, nK, nV, d, dv, page_size, num_pages, eps, status, whole, temp_coef,
-                  temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag, v_norm, v_mode, v_lambda, v_first);
-    else
-        NG_LAUNCH((qkv_prep_kernel<float>), grid, MA_THREADS, smem, stream, (const float*)qkv, (float*)q_out, qw, kw,
-                  inv_freq, rot_dims, (float*)k_pages, (float*)v_pages, table, table_stride, positions, row_entry, nQ, nK, nV,
-                  d, dv, page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm, v_is_k, rot_mag, v_norm, v_mode, v_lambda, v_first);
+#define PREP_LAUNCH(TT, OWN)                                                                                           \
+    NG_LAUNCH((qkv_prep_kernel<TT, OWN>), grid, MA_THREADS, smem, stream, (const TT*)qkv, (TT*)q_out, qw, kw, inv_freq, \
+              rot_dims, (TT*)k_pages, (TT*)v_pages, table, table_stride, positions, row_entry, nQ, nK, nV, d, dv,      \
+              page_size, num_pages, eps, status, whole, temp_coef, temp_every, ld, half_pairing, unit_norm, v_is_k,    \
+              rot_mag, v_norm, v_mode, v_lambda, v_first)
+    const bool own_v = (v_norm || v_mode) && nV > 0;
+    if (act_bf16) {
+        if (own_v) PREP_LAUNCH(__nv_bfloat16, true);
+        else PREP_LAUNCH(__nv_bfloat16, false);
+    } else {
+        if (own_v) PREP_LAUNCH(float, true);
+        else PREP_LAUNCH(float, false);
+    }
     return ng_launch_status();
 }
 

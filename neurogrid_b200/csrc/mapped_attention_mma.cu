@@ -102,8 +102,19 @@ __device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t&
 // take different keys of every tile (each keeps a softmax state of its own; merged in warp order at the end), and
 // instead of the finished heads the block leaves each run's state (maximum, sum, weighted values) for the kernel that
 // merges runs.
+template <int M>
+constexpr size_t smem_bytes() {
+    constexpr size_t ROWS = (WARPS / M) * 16;
+    constexpr size_t tiles = (M * ROWS * QP + 2 * ((size_t)M * KT * KP + (size_t)KT * VP)) * sizeof(bf16);
+    constexpr size_t epi = M * ROWS * QP * sizeof(bf16) + (M * ROWS > 64 ? M * ROWS : 64) * DV * sizeof(float);
+    return tiles > epi ? tiles : epi;
+}
+// blocks of an SM that its shared memory holds (227 KB, 1 KB of each block's own): the registers are shared out to as many
+template <int M>
+constexpr int blocks_per_sm() { return smem_bytes<M>() + 4096 <= 227 * 1024 / 3 ? 3 : 2; }
+
 template <int M, bool GROUP>
-__global__ void __launch_bounds__(THREADS, 3)
+__global__ void __launch_bounds__(THREADS, blocks_per_sm<M>())
 mapped_attention_mma_kernel(const MmaParams p) {
     constexpr int ROWS = (WARPS / M) * 16;               // rows of a block
     constexpr int PARTS = GROUP ? WARPS / M : 1;         // warps that share a tile's keys
@@ -442,9 +453,7 @@ mapped_attention_mma_kernel(const MmaParams p) {
 template <int M, bool GROUP>
 static int mma_launch(const MmaParams& p, int n_entries, int max_q, cudaStream_t stream) {
     constexpr int ROWS = (WARPS / M) * 16;
-    const size_t tiles = ((size_t)M * ROWS * QP + 2 * ((size_t)M * KT * KP + (size_t)KT * VP)) * sizeof(bf16);
-    const size_t epi = (size_t)M * ROWS * QP * sizeof(bf16) + (size_t)(M * ROWS > 64 ? M * ROWS : 64) * DV * sizeof(float);
-    const size_t smem = tiles > epi ? tiles : epi;
+    constexpr size_t smem = smem_bytes<M>();
     static bool attr = false;
     if (!attr) {
         if (cudaFuncSetAttribute(mapped_attention_mma_kernel<M, GROUP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)

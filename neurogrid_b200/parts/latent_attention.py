@@ -16,8 +16,8 @@ class LatentAttention:
     """c_q = rmsnorm(W_dq x), q_h = W_uq,h c_q;  c = rmsnorm(W_dkv x), k_h = W_uk,h c, v_h = W_uv,h c;
     out = W_o concat_h( sigmoid(W_g x)_h * softmax(q_h k_h^T * scale) v_h ) over a window; no positions.
 
-    Only c is cached (pages without a value half, one "head" of kv_rank columns, padded to a multiple
-    of 16 with zeros).  The expansions are folded into the neighbouring matrices when the weights are
+    Only c is cached (pages without a value half, one "head" of kv_rank columns, padded with zeros to a multiple
+    of 16 or 32).  The expansions are folded into the neighbouring matrices when the weights are
     bound (in float64, rounded once to the compute dtype):
         q_h . k_h = (W_uk,h^T W_uq,h c_q) . c        -> one matrix [heads * rank, q_rank] makes the queries
         W_o,h (g_h * W_uv,h sum_j p_j c_j)           -> one matrix [hidden, heads * rank] ends the mixer
@@ -45,7 +45,9 @@ class LatentAttention:
         self.by_element = getattr(spec, "gate", "head") == "element"
         if not owns_cache and not self.rope and not self.by_element:
             raise ValueError("a latent attention layer of this form keeps its own cache")
-        self.rank_p = -(-(spec.kv_rank + self.rope) // 16) * 16
+        # a cached row, padded with zeros: in sixteens, or to what the tensor-core core takes
+        in_step = lambda step: -(-(spec.kv_rank + self.rope) // step) * step
+        self.rank_p = in_step(32) if ops.latent_core_mma_takes(spec.n_heads, in_step(32), dtype) else in_step(16)
         self.n_gate = spec.n_heads * spec.value_dim if self.by_element else 0 if spec.gate == "none" else spec.n_heads
         self.position = registry.build("position", spec.position, device=device) if self.rope else None
         self.w_down = self.w_q = self.w_out = self.w_uv = self.dq_norm = self.dkv_norm = None
@@ -139,7 +141,17 @@ class LatentAttention:
         if self.rope:
             ops.latent_rope_q(q, ctx.positions, ctx.row_entry, pa.inv_freq, H, s.kv_rank, pa.half_pairing, rot_mag=pa.magnitude)
         o = ctx.ws.buf("lat_o", n, H * rp, self.dtype)
-        head_gate = None if self.by_element else gate
+        self.attend(q, cache, ctx, o, None if self.by_element else gate)
+        if self.by_element:                     # expand every head's weighted latent to its values, gate them, project
+            a = ctx.ws.buf("lat_heads", n, H * s.value_dim, self.dtype)
+            ops.head_up_gate(o, self.w_uv, gate, a)
+            return ops.linear_to_residual(a, self.w_out, None, ctx.ws, "mixer_out", residual=ctx.residual)
+        return ops.linear_to_residual(o, self.w_out, None, ctx.ws, "mixer_out", residual=ctx.residual)
+
+    def attend(self, q, cache, ctx, o, head_gate=None):
+        """The attention core over the latent pages: q, o [N, n_heads * rank_p]; ``head_gate``: a gate per head or None."""
+        s = self.spec
+        n, H, rp = q.shape[0], s.n_heads, self.rank_p
         if n > self.SPLIT_MAX_ROWS and ops.latent_core_mma_takes(H, rp, self.dtype):
             ops.latent_core_mma(q, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, head_gate, o, H, s.window,
                                 s.softmax_scale)
@@ -159,9 +171,4 @@ class LatentAttention:
             ops.attention_generic(q, cache.k_pages, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, o,
                                   H, s.window, s.softmax_scale)
             if head_gate is not None:
-                ops.head_gate(o, gate, H)
-        if self.by_element:                     # expand every head's weighted latent to its values, gate them, project
-            a = ctx.ws.buf("lat_heads", n, H * s.value_dim, self.dtype)
-            ops.head_up_gate(o, self.w_uv, gate, a)
-            return ops.linear_to_residual(a, self.w_out, None, ctx.ws, "mixer_out", residual=ctx.residual)
-        return ops.linear_to_residual(o, self.w_out, None, ctx.ws, "mixer_out", residual=ctx.residual)
+                ops.head_gate(o, head_gate, H)

@@ -91,3 +91,15 @@ def dodilix_dirs(tmp_path_factory):
         out[name + "_calm"] = dodilix_models.write_model(cfg, seed, str(tmp_path_factory.mktemp(f"dodilix_{name}c")),
                                                          same_experts=True)
     return out
+
+
+@pytest.fixture(scope="session")
+def pepulix_dirs(tmp_path_factory):
+    """Model folders for the tiny Pepulix configurations; "<name>_calm" has routers that hardly look at the token, for
+    comparisons in bfloat16."""
+    import pepulix_models
+    out = {}
+    for name, (cfg, seed) in pepulix_models.CONFIGS.items():
+        out[name] = pepulix_models.write_model(cfg, seed, str(tmp_path_factory.mktemp(f"pepulix_{name}")))
+        out[name + "_calm"] = pepulix_models.write_model(cfg, seed, str(tmp_path_factory.mktemp(f"pepulix_{name}c")), calm=True)
+    return out

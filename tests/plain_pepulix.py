@@ -101,7 +101,7 @@ def attention(h, w, pre, m, eps, v_first=None):
 # ------------------------------------------------------------------------------------------------ latent attention
 def latent_attention(h, w, pre, m, eps):
     T = h.shape[0]
-    H, d, r, dv, rank = m["heads"], m["dim"], m["rot_dim"], m["vdim"], m["kv_rank"]
+    H, d, r, dv, rank = m["heads"], m["dim"], m.get("rot_dim", 0), m["vdim"], m["kv_rank"]
     cq = rms_norm(h @ w[pre + "dq"].T, w[pre + "dq.norm"], eps)
     q = (cq @ w[pre + "uq"].T).view(T, H, d + r)
     down = h @ w[pre + "dkv"].T
