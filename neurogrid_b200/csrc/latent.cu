@@ -302,34 +302,54 @@ latent_core_kernel(const T* __restrict__ q, const T* __restrict__ pages, const i
     }
 }
 
-// merges the runs of a (row, head) in ascending order: a warp each
+// merges the runs of a (row, head) in ascending order, a block each: the runs' factors once, then a thread per column
+#define LC_MAX_SPLITS 64
 template <typename T>
-__global__ void latent_merge_kernel(const float* __restrict__ partial, const float* __restrict__ gate,
-                                    const int* __restrict__ row_entry, T* __restrict__ out, int n_rows, int nH, int rp,
-                                    int n_splits) {
+__global__ void __launch_bounds__(256)
+latent_merge_kernel(const float* __restrict__ partial, const float* __restrict__ gate, const int* __restrict__ row_entry,
+                    T* __restrict__ out, int nH, int rp, int n_splits) {
+    __shared__ float f_s[LC_MAX_SPLITS];
+    __shared__ float scale_s;
     ng_pdl_trigger();
     ng_pdl_wait();
-    const int w = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    if (w >= n_rows * nH) return;
-    const int row = w / nH;
+    const int row = blockIdx.x, w = row * nH + blockIdx.y, lane = threadIdx.x & 31;
     if (row_entry[row] < 0) return;                 // the core wrote zeros there
     const float* src = partial + (size_t)w * n_splits * (rp + 2);
-    float M = -INFINITY;
-    for (int s = 0; s < n_splits; ++s) M = fmaxf(M, src[(size_t)s * (rp + 2) + rp]);
-    float L = 0.f;
-    for (int s = 0; s < n_splits; ++s) {
-        const float ms = src[(size_t)s * (rp + 2) + rp];
-        if (ms > -INFINITY) L += src[(size_t)s * (rp + 2) + rp + 1] * expf(ms - M);
-    }
-    const float f = (L > 0.f ? 1.f / L : 0.f) * (gate ? gate[w] : 1.f);
-    for (int d = lane; d < rp; d += 32) {
-        float a = 0.f;
-        for (int s = 0; s < n_splits; ++s) {
+    if (threadIdx.x < 32) {
+        float M = -INFINITY, L = 0.f;
+        for (int s = lane; s < n_splits; s += 32) M = fmaxf(M, src[(size_t)s * (rp + 2) + rp]);
+        M = ng_warp_max(M);
+        for (int s = lane; s < n_splits; s += 32) {
             const float ms = src[(size_t)s * (rp + 2) + rp];
-            if (ms > -INFINITY) a += src[(size_t)s * (rp + 2) + d] * expf(ms - M);
+            const float f = ms > -INFINITY ? expf(ms - M) : 0.f;
+            f_s[s] = f;
+            L += src[(size_t)s * (rp + 2) + rp + 1] * f;
         }
-        ng_st(out + (size_t)w * rp + d, a * f);
+        L = ng_warp_sum(L);
+        if (lane == 0) scale_s = (L > 0.f ? 1.f / L : 0.f) * (gate ? gate[w] : 1.f);
     }
+    __syncthreads();
+    for (int d = threadIdx.x; d < rp; d += blockDim.x) {
+        float a = 0.f;
+#pragma unroll 8
+        for (int s = 0; s < n_splits; ++s) a = fmaf(src[(size_t)s * (rp + 2) + d], f_s[s], a);
+        ng_st(out + (size_t)w * rp + d, a * scale_s);
+    }
+}
+
+// partial: float32 [n_rows, nH, n_splits, rp + 2] (weighted latents, maximum, sum); rows of no entry stay as they are
+NG_EXPORT int ng_latent_merge(const float* partial, const float* gate, const int* row_entry, void* out, int n_rows, int nH,
+                              int rp, int n_splits, int act_bf16, cudaStream_t stream) {
+    if (n_rows <= 0) return NG_OK;
+    if (!partial || nH <= 0 || nH > 65535 || rp <= 0 || n_splits < 1 || n_splits > LC_MAX_SPLITS) return NG_BAD_SIZE;
+    const dim3 grid(n_rows, nH);
+    const int threads = rp <= 64 ? 64 : rp <= 128 ? 128 : 256;
+    if (act_bf16)
+        NG_LAUNCH((latent_merge_kernel<__nv_bfloat16>), grid, threads, 0, stream, partial, gate, row_entry, (__nv_bfloat16*)out,
+                  nH, rp, n_splits);
+    else
+        NG_LAUNCH((latent_merge_kernel<float>), grid, threads, 0, stream, partial, gate, row_entry, (float*)out, nH, rp, n_splits);
+    return ng_launch_status();
 }
 
 // q, out: [n_rows, nH*rp]; pages: [num_pages, 1, page_size, rp]; gate: float32 [n_rows, nH] or null.
@@ -371,15 +391,7 @@ NG_EXPORT int ng_latent_core(const void* q, const void* pages, const int* table,
     } else {
         if (hpw == 1) LC_BY_J(float, 1) else if (hpw == 2) LC_BY_J(float, 2) else LC_BY_J(float, 4)
     }
-    if (n_splits > 1) {
-        const unsigned blocks = (unsigned)(((size_t)n_rows * nH + 7) / 8);
-        if (act_bf16)
-            NG_LAUNCH((latent_merge_kernel<__nv_bfloat16>), blocks, 256, 0, stream, (const float*)partial, gate, row_entry,
-                      (__nv_bfloat16*)out, n_rows, nH, rp, n_splits);
-        else
-            NG_LAUNCH((latent_merge_kernel<float>), blocks, 256, 0, stream, (const float*)partial, gate, row_entry,
-                      (float*)out, n_rows, nH, rp, n_splits);
-    }
+    if (n_splits > 1) return ng_latent_merge(partial, gate, row_entry, out, n_rows, nH, rp, n_splits, act_bf16, stream);
     return ng_launch_status();
 }
 

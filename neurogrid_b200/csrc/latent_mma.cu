@@ -1,4 +1,4 @@
-// Latent attention core for long steps (bfloat16) on the tensor cores, with float32 scores, weights and sums.
+// Latent attention core for bfloat16 steps on the tensor cores, with float32 scores, weights and sums.
 //
 // Every head of a row reads the same latent pages as keys and as values, so the heads of ONE row are the 16
 // rows of an m16n8k16 tile: a warp takes a row, copies 32 latents at a time into shared memory (cp.async, a tile ahead),
@@ -11,7 +11,8 @@
 // The head's gate multiplies the result in the store.  Up to 16 heads (rows of the tile past the heads are zero; with
 // eight heads or fewer the tile's lower half takes the next query row),
 // rank a multiple of 32 fixed at compile time (-DNG_LAT_RANK).  Keys are walked in ascending order from the
-// window's first key: a row's result does not depend on the cut or the batch.
+// window's first key: a row's result does not depend on the cut or the batch.  Steps of few rows cut every row's keys into
+// runs, a warp each, whose states (weighted latents, maximum, sum) the merge kernel of latent.cu puts together.
 #include "ng_common.cuh"
 
 #ifndef NG_LAT_RANK
@@ -71,12 +72,14 @@ __device__ __forceinline__ void lm_split3(float x, float y, uint32_t& hi, uint32
 // PAIR (models of up to eight heads): the tile's lower eight rows are the heads of the NEXT query row, so no half of
 // a tile is empty.  Two rows share their key tiles when they are neighbours of one request (same entry, positions p and
 // p + 1); otherwise the warp takes them one after the other, each in the upper half.
-template <bool PAIR>
+// SPLIT (not with PAIR): blockIdx.y names the run of keys, and the state goes to `partial` [row, head, run, rank + 2].
+template <bool PAIR, bool SPLIT>
 __global__ void __launch_bounds__(LM_WARPS * 32)
 latent_core_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ pages, const int* __restrict__ table,
                        int table_stride, const int* __restrict__ positions, const int* __restrict__ row_entry,
                        const float* __restrict__ gate, bf16* __restrict__ out, int n_rows, int nH, int page_size,
-                       int num_pages, int window, float scale) {
+                       int num_pages, int window, float scale, int n_splits, float* __restrict__ partial) {
+    static_assert(!(PAIR && SPLIT), "runs go with one row a tile");
     extern __shared__ __align__(16) unsigned char lm_smem[];
     ng_pdl_trigger();
     ng_pdl_wait();
@@ -99,14 +102,20 @@ latent_core_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ page
     bf16* orow = out + (size_t)row * nH * LM_R;
     const int entry = row_entry[row];
     if (entry < 0) {
-        for (int i = lane; i < nH * LM_R; i += 32) orow[i] = __float2bfloat16_rn(0.f);
+        if (!SPLIT || blockIdx.y == 0)
+            for (int i = lane; i < nH * LM_R; i += 32) orow[i] = __float2bfloat16_rn(0.f);
         continue;
     }
     const int pos = positions[row];
-    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    int lo = window > 0 ? max(0, pos - window + 1) : 0;
     const int pos1 = row1 >= 0 ? pos + 1 : pos;            // the lower half's last and first visible key
     const int lo1 = PAIR ? (window > 0 ? max(0, pos1 - window + 1) : 0) : lo;
-    const int pos_hi = pos1;                               // the last key any row of the tile sees
+    int pos_hi = pos1;                                     // the last key any row of the tile sees
+    if (SPLIT) {                                           // ... of this run (an empty run: below its first)
+        const int tiles = (pos - lo + LM_TILE) / LM_TILE, per = (tiles + n_splits - 1) / n_splits;
+        lo += (int)blockIdx.y * per * LM_TILE;
+        pos_hi = min(pos, lo + per * LM_TILE - 1);
+    }
     const int* trow = table + (size_t)entry * table_stride;
 
     // the queries as A fragments: rows quad (upper half) and quad + 8 (lower half), all of the latent's columns
@@ -152,7 +161,7 @@ latent_core_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ page
         lm_cp_commit();
     };
     __syncwarp();                                              // (a second pass: the tiles of the first are done with)
-    stage(lo, bufs);
+    if (!SPLIT || lo <= pos_hi) stage(lo, bufs);
     int it = 0;
     for (int k0 = lo; k0 <= pos_hi; k0 += LM_TILE, ++it) {
         const int n = min(LM_TILE, pos_hi + 1 - k0);
@@ -257,6 +266,19 @@ latent_core_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ page
     l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if (SPLIT) {
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const int h = quad + 8 * half;
+            if (h >= nH) break;
+            float* dst = partial + (((size_t)row * nH + h) * n_splits + blockIdx.y) * (LM_R + 2);
+#pragma unroll
+            for (int t = 0; t < LM_R / 8; ++t)
+                *reinterpret_cast<float2*>(dst + t * 8 + tq * 2) = make_float2(o[t][2 * half], o[t][2 * half + 1]);
+            if (tq == 0) *reinterpret_cast<float2*>(dst + LM_R) = half ? make_float2(m1, l1) : make_float2(m0, l0);
+        }
+        continue;
+    }
     // where the two halves' results go: (row, head quad) and, lower half, (row, head quad + 8) or (the next row, head quad)
     const int h0 = quad, h1 = PAIR ? quad : quad + 8;
     const int out_row1 = PAIR ? row1 : row;
@@ -273,29 +295,33 @@ latent_core_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ page
     }
 }
 
-// q, out: bfloat16 [n_rows, nH * NG_LAT_RANK]; pages: bfloat16 [num_pages, 1, page_size, NG_LAT_RANK]; gate float32 or null
+// q, out: bfloat16 [n_rows, nH * NG_LAT_RANK]; pages: bfloat16 [num_pages, 1, page_size, NG_LAT_RANK]; gate float32 or null.
+// n_splits > 1: runs of keys, their states to `partial` (float32 [n_rows, nH, n_splits, NG_LAT_RANK + 2]); out then gets only
+// the zeros of rows of no entry, and the gate is left to the merge.
 NG_EXPORT int ng_latent_core_mma(const void* q, const void* pages, const int* table, int table_stride, const int* positions,
                                  const int* row_entry, const float* gate, void* out, int n_rows, int nH, int rp,
-                                 int page_size, int num_pages, int window, float scale, cudaStream_t stream) {
+                                 int page_size, int num_pages, int window, float scale, int n_splits, float* partial,
+                                 cudaStream_t stream) {
     if (n_rows <= 0) return NG_OK;
-    if (rp != LM_R || nH <= 0 || nH > 16 || page_size <= 0) return NG_BAD_SIZE;
+    if (rp != LM_R || nH <= 0 || nH > 16 || page_size <= 0 || n_splits < 1 || n_splits > 65535 ||
+        (n_splits > 1 && (!partial || ((uintptr_t)partial & 7))))
+        return NG_BAD_SIZE;
     const size_t smem = (size_t)LM_WARPS * 2 * LM_TILE * LM_LD * sizeof(bf16);
     static bool configured = false;
     if (!configured) {
-        if (cudaFuncSetAttribute(latent_core_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
-            cudaFuncSetAttribute(latent_core_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+        if (cudaFuncSetAttribute(latent_core_mma_kernel<false, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(latent_core_mma_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
+            cudaFuncSetAttribute(latent_core_mma_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
             return NG_LAUNCH_FAILED;
         configured = true;
     }
-    if (nH <= 8) {                  // two query rows a tile
-        const int units = (n_rows + 1) / 2;
-        NG_LAUNCH((latent_core_mma_kernel<true>), (units + LM_WARPS - 1) / LM_WARPS, LM_WARPS * 32, smem, stream, (const bf16*)q,
-                  (const bf16*)pages, table, table_stride, positions, row_entry, gate, (bf16*)out, n_rows, nH, page_size,
-                  num_pages, window, scale);
-    } else {
-        NG_LAUNCH((latent_core_mma_kernel<false>), (n_rows + LM_WARPS - 1) / LM_WARPS, LM_WARPS * 32, smem, stream, (const bf16*)q,
-                  (const bf16*)pages, table, table_stride, positions, row_entry, gate, (bf16*)out, n_rows, nH, page_size,
-                  num_pages, window, scale);
-    }
+#define LM_LAUNCH(PP, SS, BLOCKS)                                                                                      \
+    NG_LAUNCH((latent_core_mma_kernel<PP, SS>), (BLOCKS), LM_WARPS * 32, smem, stream, (const bf16*)q, (const bf16*)pages, \
+              table, table_stride, positions, row_entry, gate, (bf16*)out, n_rows, nH, page_size, num_pages, window,   \
+              scale, n_splits, partial)
+    const unsigned row_blocks = (unsigned)((n_rows + LM_WARPS - 1) / LM_WARPS);
+    if (n_splits > 1) LM_LAUNCH(false, true, dim3(row_blocks, n_splits));
+    else if (nH <= 8) LM_LAUNCH(true, false, dim3(((n_rows + 1) / 2 + LM_WARPS - 1) / LM_WARPS));      // two query rows a tile
+    else LM_LAUNCH(false, false, dim3(row_blocks));
     return ng_launch_status();
 }

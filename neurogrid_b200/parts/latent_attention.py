@@ -24,7 +24,7 @@ class LatentAttention:
     so the attention core is a multi-query attention in which every head reads the latent pages both as
     keys and as values: a block per row stages each tile of latents once for all heads.  Scores, softmax
     weights and their sum with the values are float32, keys are walked in ascending order, and the two
-    norms and the gate are float32 too.  Long bfloat16 steps run the core on the tensor cores with the heads
+    norms and the gate are float32 too.  bfloat16 steps run the core on the tensor cores with the heads
     of a row as the rows of an MMA tile (exact products, float32 sums; the weights as three bfloat16 terms).
 
     With a rotated key part (``spec.rope_dim`` r): a cached row is [c | rotated key part | zeros], a head's query
@@ -37,7 +37,8 @@ class LatentAttention:
 
     graph_safe = True      # launches depend on device data and on launch-time constants only
     SPLIT_MAX_ROWS = 32    # steps of up to this many rows cut each row's keys into runs
-    MAX_SPLITS = 16
+    MAX_SPLITS = 32
+    MMA_RUNS = 512         # ... rows * runs on the tensor cores, where a run is a warp's
 
     def __init__(self, spec, *, dtype, device, owns_cache=True):
         self.spec, self.dtype, self.device, self.owns_cache = spec, dtype, device, owns_cache
@@ -152,21 +153,20 @@ class LatentAttention:
         """The attention core over the latent pages: q, o [N, n_heads * rank_p]; ``head_gate``: a gate per head or None."""
         s = self.spec
         n, H, rp = q.shape[0], s.n_heads, self.rank_p
-        if n > self.SPLIT_MAX_ROWS and ops.latent_core_mma_takes(H, rp, self.dtype):
-            ops.latent_core_mma(q, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, head_gate, o, H, s.window,
-                                s.softmax_scale)
-        elif ops.latent_core_takes(H, rp):
-            # a step of few rows has too few blocks for the GPU: every row's keys are cut into runs, a block each
+        # a step of few rows has too few blocks for the GPU: every row's keys are cut into runs, each worked on by itself
+        mma = ops.latent_core_mma_takes(H, rp, self.dtype)
+        if mma or ops.latent_core_takes(H, rp):
             n_splits = 1
             if n <= self.SPLIT_MAX_ROWS:
                 longest = s.window or cache.table.shape[1] * cache.k_pages.shape[2]
-                n_splits = max(1, min(self.MAX_SPLITS, 128 // n, longest // 64))
+                n_splits = max(1, min(self.MAX_SPLITS, (self.MMA_RUNS if mma else 128) // n, longest // 64))
             partial = None
             if n_splits > 1:
                 partial = ctx.ws.flat(f"lat_partial_{H}x{rp}", ops.latent_core_partial_floats(n, H, rp, n_splits), torch.float32,
                                       reserve=ops.latent_core_partial_floats(self.SPLIT_MAX_ROWS, H, rp, self.MAX_SPLITS))
-            ops.latent_core(q, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, head_gate, o, H, s.window,
-                            s.softmax_scale, n_splits, partial)
+            core = ops.latent_core_mma if mma else ops.latent_core
+            core(q, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, head_gate, o, H, s.window, s.softmax_scale,
+                 n_splits, partial)
         else:                                   # very many heads or a very wide latent: the plain kernel, then the gate
             ops.attention_generic(q, cache.k_pages, cache.k_pages, cache.table, ctx.positions, ctx.row_entry, o,
                                   H, s.window, s.softmax_scale)

@@ -16,6 +16,7 @@ def pytest_configure(config):
 
 def pytest_collection_modifyitems(config, items):
     import torch
+    torch.set_num_threads(min(8, torch.get_num_threads()))     # the oracles' tensors are small: more threads cost more than they bring
     if torch.cuda.is_available():
         return
     skip = pytest.mark.skip(reason="no CUDA device")

@@ -248,12 +248,47 @@ def test_latent_rows_and_queries_with_a_rescaled_rotation(dtype, H, rank, rot):
     assert rel_err(q, want.reshape(T, -1)) < TOL[dtype] and int(ctx.status.item()) == 0
 
 
+@pytest.mark.parametrize("H,rp", [(8, 64), (12, 32), (5, 256), (16, 160), (1, 96)])
+@pytest.mark.parametrize("window", [None, 70])
+@pytest.mark.parametrize("n_splits", [2, 7, 32])
+def test_latent_core_in_runs_of_keys(H, rp, window, n_splits):
+    """Rows of several requests, their keys cut into runs (more runs than some rows have tiles), with one key that towers
+    over hundreds, padding rows among them; a gate per head."""
+    ps, T = 16, 700
+    g = torch.Generator().manual_seed(3)
+    n_pages = 2 * (-(-T // ps)) + 4
+    pages = (0.5 * torch.randn(n_pages, 1, ps, rp, generator=g)).to(torch.bfloat16)
+    order = torch.randperm(n_pages, generator=g)[: 2 * (-(-T // ps))].view(2, -1)
+    table = torch.cat([order, torch.full((2, 2), -1)], 1).to(torch.int32)
+    pos = [0, 31, 32, 33, 699, 5, 300, 64, 640]
+    entry = [0, 1, 0, 1, 0, -1, 1, 0, 1]
+    q = (0.5 * torch.randn(len(pos), H * rp, generator=g)).to(torch.bfloat16)
+    far = pages[table[0, 640 // ps].long(), 0, 640 % ps]
+    q[4] = (4.0 * far / far.float().norm()).repeat(H).to(torch.bfloat16) + 0.1 * q[4]      # row 4 looks for key 640 of request 0
+    pages[table[0, 640 // ps].long(), 0, 640 % ps] = 4 * far
+    gate = torch.rand(len(pos), H, generator=g)
+    i32 = lambda x: torch.tensor(x, dtype=torch.int32)
+    want = torch.zeros(len(pos), H, rp, dtype=F64)
+    for r, (p, e) in enumerate(zip(pos, entry)):
+        if e < 0:
+            continue
+        keys = torch.arange(max(0, p - window + 1) if window else 0, p + 1)
+        C = pages[table[e, keys // ps].long(), 0, keys % ps].double()
+        w = torch.softmax(q[r].double().view(H, rp) @ C.T * 0.4, -1)
+        want[r] = (w @ C) * gate[r].double()[:, None]
+    out = torch.full((len(pos), H * rp), 7.0, dtype=torch.bfloat16, device=DEV)
+    partial = torch.full((ops().latent_core_partial_floats(len(pos), H, rp, n_splits),), float("nan"), device=DEV)
+    ops().latent_core_mma(q.to(DEV), pages.to(DEV), table.to(DEV), i32(pos).to(DEV), i32(entry).to(DEV), gate.to(DEV), out, H, window,
+                          0.4, n_splits, partial)
+    assert rel_err(out, want.reshape(len(pos), -1)) < 1e-2 and float(out[5].abs().max()) == 0
+
+
 def _part(spec, cls, dtype, seed, gains=None):
     part = cls(spec, dtype=dtype, device=DEV)
     g = torch.Generator().manual_seed(seed)
     w = {}
     for name, d in part.tensors().items():
-        t = torch.randn(*d.shape, generator=g)
+        t = torch.randn(d.shape, generator=g)
         t = 1 + 0.2 * t if d.init == "norm" else t if d.init == "bias" else 1.3 * t / d.shape[-1] ** 0.5
         w[name] = ((gains or {}).get(name, 1.0) * t).to(torch.bfloat16).float()
     part.bind({k: v.to(DEV) for k, v in w.items()})
