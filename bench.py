@@ -1287,13 +1287,7 @@ def dodilix_kernel_times(eng, l2, pk):
         ql, ol = rnd(rows, Hl * rp), torch.empty(rows, Hl * rp, dtype=torch.bfloat16, device=dev)
         mem(f"{tag}_latent_rope_q", timed(lambda: ops.latent_rope_q(ql, ctx.positions, ctx.row_entry, la.inv_freq, Hl, ts_.kv_rank)),
             2 * rows * Hl * lat.rope * 2)
-        if entries == 1:
-            corel = lambda: ops.latent_core_mma(ql, lp, table, ctx.positions, ctx.row_entry, None, ol, Hl, None, ts_.softmax_scale)
-        else:
-            n_splits = max(1, min(lat.MAX_SPLITS, 128 // rows, (before + 1) // 64))
-            part = torch.empty(max(1, ops.latent_core_partial_floats(rows, Hl, rp, n_splits)), device=dev)
-            corel = lambda: ops.latent_core(ql, lp, table, ctx.positions, ctx.row_entry, None, ol, Hl, None, ts_.softmax_scale,
-                                            n_splits, part)
+        corel = lambda: lat.attend(ql, PagedView(lp, None, table), ctx, ol)
         corel()
         torch.cuda.synchronize()
         pairs = sum(t + 1 for t in range(rows)) if entries == 1 else rows * (before + 1)

@@ -28,46 +28,55 @@ latent_prep_kernel(const T* __restrict__ x, const float* __restrict__ wq, const 
                    const int* __restrict__ row_entry, int rq, int rkv, int rp, int nH, int page_size, int num_pages,
                    float eps, int* __restrict__ status, int rot, const float* __restrict__ inv_freq, int half_pairing,
                    float rot_mag) {
-    __shared__ float red[32];
+    __shared__ float red[2][4];
     ng_pdl_trigger();
-    ng_pdl_wait();
-    const int row = blockIdx.x;
+    // what the step's host copy brought is read before the wait: the row's place, the angles of its first pairs
+    const int row = blockIdx.x, tid = threadIdx.x;
     const int entry = row_entry[row];
+    const int pos = positions[row];
+    int page = -1;
+    if (entry >= 0 && rkv > 0 && pos >= 0) page = table[(size_t)entry * table_stride + pos / page_size];
+    const bool place = page >= 0 && page < num_pages;
+    float sn = 0.f, cs = 0.f;
+    if (place && tid < rot / 2) sincosf((float)pos * inv_freq[tid], &sn, &cs);
+    ng_pdl_wait();
     if (entry < 0) return;
-    const T* xr = x + (size_t)row * (rq + rkv + rot + nH);
-    float ss = 0.f;
-    for (int i = threadIdx.x; i < rq; i += blockDim.x) {
+    const T* xr = ng_after_wait(x) + (size_t)row * (rq + rkv + rot + nH);
+    // both sums of squares in one pass and one meeting of the block
+    float s1 = 0.f, s2 = 0.f;
+#pragma unroll 4
+    for (int i = tid; i < rq; i += 128) {
         const float v = ng_ld(xr + i);
-        ss += v * v;
+        s1 = fmaf(v, v, s1);
     }
-    ss = ng_block_sum(ss, red);
-    const float r1 = rsqrtf(ss / (float)rq + eps);
-    for (int i = threadIdx.x; i < rq; i += blockDim.x) ng_st(cq_out + (size_t)row * rq + i, ng_ld(xr + i) * r1 * wq[i]);
+#pragma unroll 4
+    for (int i = tid; i < rkv; i += 128) {
+        const float v = ng_ld(xr + rq + i);
+        s2 = fmaf(v, v, s2);
+    }
+    s1 = ng_warp_sum(s1);
+    s2 = ng_warp_sum(s2);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = s1; red[1][tid >> 5] = s2; }
+    __syncthreads();
+    const float r1 = rsqrtf((red[0][0] + red[0][1] + red[0][2] + red[0][3]) / (float)rq + eps);
+#pragma unroll 4
+    for (int i = tid; i < rq; i += 128) ng_st(cq_out + (size_t)row * rq + i, ng_ld(xr + i) * r1 * wq[i]);
     if (rkv > 0) {
-        ss = 0.f;
-        for (int i = threadIdx.x; i < rkv; i += blockDim.x) {
-            const float v = ng_ld(xr + rq + i);
-            ss += v * v;
-        }
-        ss = ng_block_sum(ss, red);
-        const float r2 = rsqrtf(ss / (float)rkv + eps);
-        const int pos = positions[row];
-        const int page = pos >= 0 ? table[(size_t)entry * table_stride + pos / page_size] : -1;
-        if (page < 0 || page >= num_pages) {
-            if (threadIdx.x == 0) atomicOr(status, NG_STATUS_BAD_PAGE);
+        const float r2 = rsqrtf((red[1][0] + red[1][1] + red[1][2] + red[1][3]) / (float)rkv + eps);
+        if (!place) {
+            if (tid == 0) atomicOr(status, NG_STATUS_BAD_PAGE);
         } else {
             T* dst = pages + ((size_t)page * page_size + (pos % page_size)) * rp;
-            for (int i = threadIdx.x; i < rp; i += blockDim.x)
+#pragma unroll 4
+            for (int i = tid; i < rp; i += 128)
                 if (i < rkv || i >= rkv + rot) ng_st(dst + i, i < rkv ? ng_ld(xr + rq + i) * r2 * wkv[i] : 0.f);
             const T* kr = xr + rq + rkv;
-            for (int i = threadIdx.x; i < rot / 2; i += blockDim.x) {
+            for (int i = tid; i < rot / 2; i += 128) {
                 const int c1 = half_pairing ? i : 2 * i, c2 = half_pairing ? i + rot / 2 : 2 * i + 1;
-                float sn, cs;
-                sincosf((float)pos * inv_freq[i], &sn, &cs);
-                sn *= rot_mag; cs *= rot_mag;
-                const float a = ng_ld(kr + c1), b = ng_ld(kr + c2);
-                ng_st(dst + rkv + c1, a * cs - b * sn);
-                ng_st(dst + rkv + c2, b * cs + a * sn);
+                if (i != tid) sincosf((float)pos * inv_freq[i], &sn, &cs);
+                const float a = ng_ld(kr + c1), b = ng_ld(kr + c2), sm = sn * rot_mag, cm = cs * rot_mag;
+                ng_st(dst + rkv + c1, a * cm - b * sm);
+                ng_st(dst + rkv + c2, b * cm + a * sm);
             }
         }
     }

@@ -261,29 +261,39 @@ moe_router_sigmoid_kernel(const T* __restrict__ x, const float* __restrict__ wr,
                     for (int e = g * per; e < (g + 1) * per; ++e) choice[e] = -INFINITY;
             }
         }
-        int idx[MOE_MAX_TOP];
-        float sum = 0.f;
-        for (int k = 0; k < top_k; ++k) {
-            int best = -1;
-            float bv = -INFINITY;
-            for (int e = 0; e < E; ++e) {
-                const float v = choice[e];
-                if (best < 0 || v > bv) {
-                    bool taken = false;
-                    for (int m = 0; m < k; ++m) taken |= idx[m] == e;
-                    if (!taken) { best = e; bv = v; }
-                }
-            }
-            idx[k] = best;
-            sum += z[best];
+    }
+    if (warp != 0) return;
+    __syncwarp();
+    // the first warp, one expert a round: every lane the best of its experts, then the best of the lanes; of equal choice
+    // scores the lower index
+    int mine = 0;                                // lane k: the k-th chosen expert
+    float sum = 0.f;
+    for (int k = 0; k < top_k; ++k) {
+        float bv = -INFINITY;
+        int best = E;
+        for (int e = lane; e < E; e += 32) {
+            const float v = choice[e];
+            if (v > bv || (v == bv && e < best)) { bv = v; best = e; }
         }
-        float identity = 0.f;
-        for (int k = 0; k < top_k; ++k) {
-            const float w = z[idx[k]] / (sum + 1e-20f) * route_scale;
-            if (idx[k] < n_own) out[idx[k]] = w;
-            else identity += w;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+            const int oe = __shfl_xor_sync(0xffffffffu, best, o);
+            if (ov > bv || (ov == bv && oe < best)) { bv = ov; best = oe; }
         }
-        if (n_identity) out[n_own + (wsg ? 1 : 0)] = identity;
+        best = min(best, E - 1);                 // (scores that are no numbers: some expert all the same)
+        if (lane == k) mine = best;
+        sum += z[best];
+        __syncwarp();
+        if (lane == 0) choice[best] = -INFINITY;
+        __syncwarp();
+    }
+    const float w = lane < top_k ? z[mine] / (sum + 1e-20f) * route_scale : 0.f;
+    const bool own = mine < n_own;
+    if (lane < top_k && own) out[mine] = w;
+    if (n_identity) {
+        const float identity = ng_warp_sum(own ? 0.f : w);
+        if (lane == 0) out[n_own + (wsg ? 1 : 0)] = identity;
     }
 }
 

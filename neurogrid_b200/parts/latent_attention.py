@@ -37,7 +37,7 @@ class LatentAttention:
 
     graph_safe = True      # launches depend on device data and on launch-time constants only
     SPLIT_MAX_ROWS = 32    # steps of up to this many rows cut each row's keys into runs
-    MAX_SPLITS = 32
+    MAX_SPLITS = 64
     MMA_RUNS = 512         # ... rows * runs on the tensor cores, where a run is a warp's
 
     def __init__(self, spec, *, dtype, device, owns_cache=True):
