@@ -398,7 +398,7 @@ def test_biases_in_the_products_epilogue(M, K, I):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("E,n_id,top,groups,keep,shared", [(16, 4, 3, 1, 1, False), (3, 5, 4, 1, 1, False), (1, 1, 1, 1, 1, False), (6, 2, 2, 4, 2, True), (40, 24, 8, 1, 1, False)])
+@pytest.mark.parametrize("E,n_id,top,groups,keep,shared", [(14, 6, 3, 1, 1, False), (3, 5, 4, 1, 1, False), (1, 1, 1, 1, 1, False), (6, 2, 2, 4, 2, True), (40, 24, 8, 1, 1, False)])
 def test_router_with_identity_experts(dtype, E, n_id, top, groups, keep, shared):
     rows, H = 37, 72
     x = _x((rows, H), dtype)
